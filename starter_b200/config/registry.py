@@ -34,6 +34,7 @@ class TensorNames:
     final_norm: Dict[str, str]
     layers: List[Dict[str, Dict[str, str]]] = field(default_factory=list)
     loop_step: str = ""   # the [times, hidden] table of a model whose layers run in passes
+    embedding_norm: Dict[str, str] = field(default_factory=dict)   # of a model that norms its embedded rows
 
 
 class ModelConfig:

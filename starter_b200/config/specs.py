@@ -46,12 +46,26 @@ class GroupedNormSpec:
 
 
 @dataclass(frozen=True)
+class LayerNormSpec:
+    """Layer norm over the last axis (kind "layernorm"): (x - mean) / sqrt(mean((x - mean)^2) + eps) * w + b."""
+
+    size: int
+    eps: float
+    kind: str = "layernorm"
+
+
+@dataclass(frozen=True)
 class PairRopeSpec:
     """Rotary position encoding over neighbouring columns: (2j, 2j + 1) of the first ``rotary_dim`` columns turn
-    by angle(p, j) = p * theta**(-2j / rotary_dim); angles, sines and the rotation itself are 32-bit."""
+    by angle(p, j) = p * theta**(-2j / rotary_dim); angles, sines and the rotation itself are 32-bit.  With ``factor``
+    the frequencies are stretched by wavelength as ScaledHalfRopeSpec says."""
 
     theta: float
     rotary_dim: int
+    factor: Optional[float] = None
+    original: Optional[float] = None
+    fast: Optional[float] = None
+    slow: Optional[float] = None
     kind: str = "rope_pairs"
 
 
@@ -268,6 +282,32 @@ class GLASpec:
 
 
 @dataclass(frozen=True)
+class ChannelDeltaSpec:
+    """Gated delta rule with a decay per key channel (kind "channel_delta"): per head a [head_dim, v_dim] state that
+    decays channel by channel, is corrected towards v at k, and is then read:
+
+        S <- g * S;   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q
+
+    q, k (``num_kv_heads`` heads of ``head_dim``, head h reads q/k head h // (num_heads / num_kv_heads)) and v
+    (``num_heads`` heads of ``v_dim``) pass a short causal convolution over time per channel (``taps``; not added to its
+    input) and silu; q and k are divided by sqrt(sum(x^2) + 1e-6) per head, q times head_dim**-0.5 as well;
+    beta = sigmoid(W_b h) per head; g = exp(-exp(A_log_h) softplus(W_a2 (W_a1 h) + dt_bias)) per head and key channel,
+    inner size ``decay_rank``.  Each head's o is divided by its root mean square (``norm_eps``), multiplied by a weight
+    of v_dim values that the heads share and by sigmoid(W_g2 (W_g1 h)), inner size ``gate_rank``, then projected."""
+
+    hidden_size: int
+    num_heads: int
+    num_kv_heads: int
+    head_dim: int
+    v_dim: int
+    taps: int
+    decay_rank: int
+    gate_rank: int
+    norm_eps: float
+    kind: str = "channel_delta"
+
+
+@dataclass(frozen=True)
 class LatentAttentionSpec:
     """Causal attention through low-rank latents (kind "latent_attention").
 
@@ -275,7 +315,9 @@ class LatentAttentionSpec:
     rotated] columns.  Keys and values: W_dkv h gives ``kv_rank`` columns that are normed (the latent) and ``rot_dim``
     more that are rotated and shared by all heads; a head's plain key and its value (``v_dim`` columns) are
     up-projections of the latent.  Only the latent and the rotated part are cached.  ``sink``: the softmax's
-    denominator holds one more term exp(s_h), a learned number per head with no key or value.
+    denominator holds one more term exp(s_h), a learned number per head with no key or value.  ``head_gate``: head h's
+    output is multiplied by sigmoid(W_g h)_h.  ``kv_from``: index of another latent attention layer of the same
+    ``kv_rank``, ``rot_dim`` and rotation whose cached rows this layer reads; it then has no W_dkv.
     """
 
     hidden_size: int
@@ -289,6 +331,8 @@ class LatentAttentionSpec:
     norm_eps: float
     position: Optional[Any] = None
     sink: bool = False
+    head_gate: bool = False
+    kv_from: Optional[int] = None
     kind: str = "latent_attention"
 
 
@@ -311,7 +355,7 @@ class GatedMLPSpec:
     """Dense gated feed-forward: down(act(gate(x)) * up(x)).
 
     ``activation`` "silu": silu(g) * u.  "clamped_swish": g' = min(g, limit), u' = clamp(u, -limit, limit),
-    g' * sigmoid(alpha * g') * (u' + 1)."""
+    g' * sigmoid(alpha * g') * (u' + 1).  "gelu_tanh": g / 2 (1 + tanh(sqrt(2 / pi) (g + 0.044715 g^3))) * u."""
 
     hidden_size: int
     intermediate_size: int
@@ -438,12 +482,12 @@ class LoopSpec:
 
 @dataclass(frozen=True)
 class BlockSpec:
-    """One layer: x += mixer(norm(x)); x += ff(norm(x)) for kind "prenorm"."""
+    """One layer: x += mixer(norm(x)); x += ff(norm(x)) for kind "prenorm"; ``ff`` and its norm may be absent."""
 
     mixer_norm: Any
     mixer: Any
-    ff_norm: Any
-    ff: Any
+    ff_norm: Any = None
+    ff: Any = None
     kind: str = "prenorm"
 
 
@@ -479,6 +523,9 @@ class ModelSpec:
     from the token ids and the rows' positions); None: positions enter in the mixers only.
 
     ``loop``: a run of layers that repeats (see LoopSpec); it takes the place of ``schedule`` and needs a 32-bit residual.
+
+    ``embedding_norm``: a norm of the embedded rows (its ``embed`` makes the first residual, 32-bit, from the token ids);
+    it needs a 32-bit residual.
     """
 
     hidden_size: int
@@ -494,6 +541,7 @@ class ModelSpec:
     streams: Optional[int] = None
     position_embedding: Optional[Any] = None
     loop: Optional[LoopSpec] = None
+    embedding_norm: Optional[Any] = None
 
     def execution_order(self) -> Tuple[int, ...]:
         if self.loop is not None:

@@ -38,6 +38,12 @@ class DecoderModel:
         norm_cls = part_class("norm", spec.final_norm.kind)
         self.final_norm = norm_cls(spec.final_norm,
                                    {r: load(names.final_norm[r]) for r in norm_cls.weight_shapes(spec.final_norm)}, runtime)
+        self.embedding_norm = None
+        if getattr(spec, "embedding_norm", None) is not None:
+            if not spec.residual_float32 or spec.streams is not None or spec.position_embedding is not None or spec.loop is not None \
+                    or spec.embedding_scale is not None:
+                raise ValueError("a norm of the embedded rows makes one 32-bit residual and nothing else enters there")
+            self.embedding_norm = build_part("norm", spec.embedding_norm, {r: load(n) for r, n in names.embedding_norm.items()}, runtime)
         self.position = None   # a position part that enters at the embedding
         if getattr(spec, "position_embedding", None) is not None:
             self.position = build_part("position", spec.position_embedding, {}, runtime)
@@ -84,6 +90,8 @@ class DecoderModel:
     def parts(self):
         """Every part object of the model: the final norm, each block, and what each block is made of."""
         yield self.final_norm
+        if self.embedding_norm is not None:
+            yield self.embedding_norm
         for block, block_spec in zip(self.blocks, self.spec.layers):
             yield block
             for name, _, _ in type(block).sub_parts(block_spec):
@@ -126,7 +134,9 @@ class DecoderModel:
             for pos, i in enumerate(self.order):
                 self.blocks[i].forward(ctx, stream, ctx.cache.layers[pos])
             return stream
-        if self.position is not None:
+        if self.embedding_norm is not None:
+            x = self.embedding_norm.embed(ctx, tokens, self.embedding)   # normed 32-bit rows
+        elif self.position is not None:
             x = self.position.embed(ctx, tokens, self.embedding)   # 32-bit rows with the positions' vectors added
         elif self.spec.residual_float32 and self.embedding.dtype != torch.float32:
             x = ctx.ops.embed(tokens, self.embedding, ctx.status, out_float32=True)   # the residual stays 32-bit
@@ -168,5 +178,5 @@ class DecoderModel:
         if self.spec.logit_scale is not None:
             logits = logits * self.spec.logit_scale
         if self.spec.logit_softcap is not None:
-            logits = torch.tanh(logits / self.spec.logit_softcap) * self.spec.logit_softcap
+            logits = ops.softcap(logits, self.spec.logit_softcap)
         return logits

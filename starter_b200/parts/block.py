@@ -1,4 +1,4 @@
-"""A layer's arrangement (kind "prenorm"): x += mixer(norm(x)); x += ff(norm(x)).
+"""A layer's arrangement (kind "prenorm"): x += mixer(norm(x)); x += ff(norm(x)); the feed-forward may be absent.
 
 Order of the reference's layer (OPTIMIZATION_GUIDE.md:60-69,
 engine/model.py:289-298).  Each branch leaves its output on the residual
@@ -23,10 +23,13 @@ class PreNormBlock:
     @staticmethod
     def sub_parts(spec):
         """(name, category, spec) of the parts this block is made of."""
-        return (("mixer_norm", "norm", spec.mixer_norm), ("mixer", "mixer", spec.mixer),
-                ("ff_norm", "norm", spec.ff_norm), ("ff", "ff", spec.ff))
+        parts = (("mixer_norm", "norm", spec.mixer_norm), ("mixer", "mixer", spec.mixer))
+        if spec.ff is not None:
+            parts += (("ff_norm", "norm", spec.ff_norm), ("ff", "ff", spec.ff))
+        return parts
 
     def __init__(self, spec, weights, runtime):
+        self.ff = self.ff_norm = None
         self.folds = getattr(runtime.ops, "folds", None)
         for name, category, sub in self.sub_parts(spec):
             setattr(self, name, build_part(category, sub, weights[name], runtime))
@@ -36,7 +39,8 @@ class PreNormBlock:
 
     def prepare(self, cache) -> None:
         self.mixer.prepare(cache)
-        self.ff.prepare(cache)
+        if self.ff is not None:
+            self.ff.prepare(cache)
 
     def _branch(self, ctx, stream, norm, part, *args) -> None:
         fold = None
@@ -52,7 +56,8 @@ class PreNormBlock:
 
     def forward(self, ctx, stream, layer_cache) -> None:
         self._branch(ctx, stream, self.mixer_norm, self.mixer, layer_cache)
-        self._branch(ctx, stream, self.ff_norm, self.ff)
+        if self.ff is not None:
+            self._branch(ctx, stream, self.ff_norm, self.ff)
 
 
 class ParallelBlock:

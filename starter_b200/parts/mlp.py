@@ -1,5 +1,6 @@
 """Dense gated feed-forward (kind "gated_mlp"): down(silu(gate(x)) * up(x)), or with the activation
-"clamped_swish" down(g * sigmoid(alpha g) * (u + 1)) for g = min(gate(x), limit), u = clamp(up(x), -limit, limit).
+"clamped_swish" down(g * sigmoid(alpha g) * (u + 1)) for g = min(gate(x), limit), u = clamp(up(x), -limit, limit), or
+with "gelu_tanh" the tanh form of gelu in silu's place.
 
 The reference fuses gate and up into one [2I, H] matrix, gate half first
 (engine/model.py:116, engine/kernels/swiglu.py:5-6), and rounds gate, up,
@@ -23,8 +24,8 @@ class GatedMLP:
         }
 
     def __init__(self, spec, weights, runtime):
-        if spec.activation not in ("silu", "clamped_swish"):
-            raise ValueError(f"activation {spec.activation!r} is not built; 'silu' and 'clamped_swish' are")
+        if spec.activation not in ("silu", "clamped_swish", "gelu_tanh"):
+            raise ValueError(f"activation {spec.activation!r} is not built; 'silu', 'clamped_swish' and 'gelu_tanh' are")
         self.activation = spec.activation
         if self.activation == "clamped_swish":
             if spec.limit is None or not spec.limit > 0:
@@ -45,6 +46,8 @@ class GatedMLP:
         product; with ``residual`` the result is added to that tensor instead of being returned on its own."""
         if self.activation == "clamped_swish":
             return self.ops.linear(self.ops.linear_gated_clamp(h, self.w_gate_up, self.alpha, self.limit), self.w_down)
+        if self.activation == "gelu_tanh":
+            return self.ops.linear(self.ops.linear_gated_gelu(h, self.w_gate_up), self.w_down)
         if norm is None and residual is None:
             return self.ops.linear(self.ops.linear_swiglu(h, self.w_gate_up), self.w_down)
         act = self.ops.linear_swiglu(h, self.w_gate_up, norm=norm)

@@ -96,6 +96,35 @@ class BranchRMSNorm:
         return self.ops.branch_norm_add(x, y, self.weight, self.scale, self.eps, self.dtype if want_rounded else None)
 
 
+class LayerNorm:
+    """Kind "layernorm": (x - mean) / sqrt(variance + eps) * w + b, all 32-bit, rounded once when the result is stored.  It
+    reads rows of the residual's type and hands out rows of the run's dtype; ``embed`` makes the first residual of a model
+    that norms its embedded rows: 32-bit rows straight from the token ids."""
+
+    @staticmethod
+    def weight_shapes(spec):
+        return {"weight": (spec.size,), "bias": (spec.size,)}
+
+    def __init__(self, spec, weights, runtime):
+        self.size = spec.size
+        self.eps = float(spec.eps)
+        self.weight = weights["weight"].float().contiguous()
+        self.bias = weights["bias"].float().contiguous()
+        self.ops = runtime.ops
+        self.dtype = runtime.dtype
+
+    def forward(self, x):
+        return self.ops.layernorm(x, None, self.weight, self.bias, self.eps, self.dtype)
+
+    def add_forward(self, x, delta):
+        """x += delta in place and in 32-bit, then the norm of the new x."""
+        return self.ops.layernorm(x, delta, self.weight, self.bias, self.eps, self.dtype)
+
+    def embed(self, ctx, tokens, table):
+        return self.ops.embed_layernorm(tokens, table, self.weight, self.bias, self.eps, ctx.status)
+
+
+register_part("norm", "layernorm", LayerNorm)
 register_part("norm", "rmsnorm", RMSNorm)
 register_part("norm", "branch_rmsnorm", BranchRMSNorm)
 register_part("norm", "grouped_rmsnorm", GroupedRMSNorm)

@@ -9,7 +9,8 @@ picks the class.  Every part class offers
 
 and, by category,
 
-* norm:     ``forward(x) -> y`` and ``add_forward(x, delta) -> y`` (x += delta in place, then norm);
+* norm:     ``forward(x) -> y`` and ``add_forward(x, delta) -> y`` (x += delta in place, then norm); one that a model puts
+  on its embedded rows: ``embed(ctx, tokens, table) -> 32-bit rows``;
 * position: ``prepare(n_positions)`` and ``fused_rotary()`` or ``apply(ctx, q, k)``; one that enters at the embedding:
   ``embed(ctx, tokens, table) -> 32-bit rows``;
 * conv:     ``cache_request()`` and ``forward(ctx, x, layer_cache) -> rows in the run's dtype``;

@@ -46,10 +46,29 @@ class RotaryEmbedding:
         return self.cos, self.sin, self.rotary_dim
 
 
+def stretched_frequencies(spec, device):
+    """(32-bit frequencies [rotary_dim / 2] on the device, what multiplies cosines and sines) of a rotation over the first
+    ``rotary_dim`` columns; with ``factor`` the frequencies are stretched by wavelength (see ScaledHalfRopeSpec)."""
+    dims = int(spec.rotary_dim)
+    i = torch.arange(dims // 2, dtype=torch.float64)
+    f = float(spec.theta) ** (-2.0 * i / dims)
+    magnitude = 1.0
+    if spec.factor is not None:
+        def pair_at(turns):
+            return dims * math.log(float(spec.original) / (2.0 * math.pi * float(turns))) / (2.0 * math.log(float(spec.theta)))
+        lo = max(math.floor(pair_at(spec.fast)), 0)
+        hi = min(math.ceil(pair_at(spec.slow)), dims - 1)
+        ramp = ((i - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+        f = f / float(spec.factor) * ramp + f * (1.0 - ramp)
+        magnitude = 0.1 * math.log(float(spec.factor)) + 1.0
+    return f.to(torch.float32).to(device), magnitude
+
+
 class PairRotary:
     """Kind "rope_pairs": neighbouring columns (2j, 2j + 1) turn together.  It keeps no table of sines: the kernels
     that rotate take the row's position from the step's batch, multiply it in 32-bit with the frequency
-    theta**(-2j / rotary_dim) from ``frequencies`` (32-bit, [rotary_dim / 2]) and take sine and cosine there."""
+    theta**(-2j / rotary_dim) from ``frequencies`` (32-bit, [rotary_dim / 2]; stretched by wavelength when the spec gives a
+    factor) and take sine and cosine there, times ``magnitude``."""
 
     @staticmethod
     def weight_shapes(spec):
@@ -60,8 +79,8 @@ class PairRotary:
             raise ValueError(f"rotary_dim must be positive and even, got {spec.rotary_dim}")
         self.theta = float(spec.theta)
         self.rotary_dim = int(spec.rotary_dim)
-        j = torch.arange(self.rotary_dim // 2, dtype=torch.float32)
-        self.frequencies = (torch.tensor(self.theta, dtype=torch.float32) ** (-2.0 * j / self.rotary_dim)).to(runtime.device)
+        self.halves = False     # how a pair's two columns stand: neighbours, not half the rotated part apart
+        self.frequencies, self.magnitude = stretched_frequencies(spec, runtime.device)
 
     def prepare(self, n_positions: int) -> None:
         pass
@@ -81,18 +100,8 @@ class ScaledHalfRotary:
         if dims <= 0 or dims % 2:
             raise ValueError(f"rotary_dim must be positive and even, got {spec.rotary_dim}")
         self.rotary_dim = dims
-        i = torch.arange(dims // 2, dtype=torch.float64)
-        f = float(spec.theta) ** (-2.0 * i / dims)
-        self.magnitude = 1.0
-        if spec.factor is not None:
-            def pair_at(turns):
-                return dims * math.log(float(spec.original) / (2.0 * math.pi * float(turns))) / (2.0 * math.log(float(spec.theta)))
-            lo = max(math.floor(pair_at(spec.fast)), 0)
-            hi = min(math.ceil(pair_at(spec.slow)), dims - 1)
-            ramp = ((i - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
-            f = f / float(spec.factor) * ramp + f * (1.0 - ramp)
-            self.magnitude = 0.1 * math.log(float(spec.factor)) + 1.0
-        self.frequencies = f.to(torch.float32).to(runtime.device)
+        self.halves = True
+        self.frequencies, self.magnitude = stretched_frequencies(spec, runtime.device)
 
     def prepare(self, n_positions: int) -> None:
         pass

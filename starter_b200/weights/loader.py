@@ -42,6 +42,9 @@ def expected_tensors(spec, names) -> Tuple[Dict[str, Tuple[int, ...]], Dict[str,
         if not names.loop_step:
             raise WeightsError("the architecture names no tensor for the passes' vectors")
         required[names.loop_step] = (spec.loop.times, spec.hidden_size)
+    if getattr(spec, "embedding_norm", None) is not None:
+        for role, shape in part_class("norm", spec.embedding_norm.kind).weight_shapes(spec.embedding_norm).items():
+            required[names.embedding_norm[role]] = tuple(shape)
     if len(names.layers) != len(spec.layers):
         raise WeightsError(f"{len(names.layers)} layers are named for {len(spec.layers)} layers")
     for block_spec, block_names in zip(spec.layers, names.layers):

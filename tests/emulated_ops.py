@@ -57,28 +57,37 @@ class EmulatedOps:
     def tanh(self, x):
         return torch.tanh(x.float()).to(x.dtype)
 
-    def linear_heads(self, a, w, out):
-        out.copy_(torch.einsum("rhk,hnk->rhn", a.float(), w.float()).to(out.dtype))
+    def linear_heads(self, a, w, out, gate=None):
+        res = torch.einsum("rhk,hnk->rhn", a.float(), w.float())
+        if gate is not None:
+            res = res.to(out.dtype).float() * torch.sigmoid(gate.float())[:, :, None]
+        out.copy_(res.to(out.dtype))
         return out
 
+    def gate_heads(self, a, gate):
+        return (a.float() * torch.sigmoid(gate.float())[:, :, None]).to(a.dtype)
+
     @staticmethod
-    def _turn(t, pos, freqs, rot):
-        """t [rows, heads, R] with its first ``rot`` columns rotated in neighbouring pairs."""
+    def _turn(t, pos, freqs, rot, magnitude=1.0, halves=False):
+        """t [rows, heads, R] with its first ``rot`` columns rotated in neighbouring pairs, or with ``halves`` column i with
+        column i + rot / 2."""
         if freqs is None or not rot:
             return t.clone()
         angle = pos.float()[:, None] * freqs.float()[None, :]
-        c, s = torch.cos(angle)[:, None, :], torch.sin(angle)[:, None, :]
-        a, b = t[..., 0:rot:2], t[..., 1:rot:2]
+        c, s = (torch.cos(angle) * magnitude)[:, None, :], (torch.sin(angle) * magnitude)[:, None, :]
+        first, second = (slice(0, rot // 2), slice(rot // 2, rot)) if halves else (slice(0, rot, 2), slice(1, rot, 2))
+        a, b = t[..., first], t[..., second]
         out = t.clone()
-        out[..., 0:rot:2] = a * c - b * s
-        out[..., 1:rot:2] = b * c + a * s
+        out[..., first] = a * c - b * s
+        out[..., second] = b * c + a * s
         return out
 
-    def rotate_pairs(self, ctx, src, dst, freqs, rot):
+    def rotate_pairs(self, ctx, src, dst, freqs, rot, magnitude=1.0, halves=False):
         _, pos = self._positions(ctx)
-        dst.copy_(self._turn(src.float(), pos, freqs, rot).to(dst.dtype))
+        dst.copy_(self._turn(src.float(), pos, freqs, rot, magnitude, halves).to(dst.dtype))
 
-    def latent_prepare(self, ctx, down, layer_cache, q_rank, kv_rank, rot_dim, q_norm, kv_norm, eps, freqs, rot, rows_too=False):
+    def latent_prepare(self, ctx, down, layer_cache, q_rank, kv_rank, rot_dim, q_norm, kv_norm, eps, freqs=None, rot=0, magnitude=1.0,
+                       halves=False, rows_too=False):
         dt = down.dtype
         slots, pos = self._positions(ctx)
         d = down.float()
@@ -87,8 +96,10 @@ class EmulatedOps:
             return t * torch.rsqrt((t * t).mean(-1, keepdim=True) + eps)
 
         cq = (unit(d[:, :q_rank]) * q_norm.float()).to(dt)
+        if layer_cache is None:
+            return cq
         latent = unit(d[:, q_rank:q_rank + kv_rank]) * kv_norm.float()
-        shared = self._turn(d[:, None, q_rank + kv_rank:], pos, freqs, rot)[:, 0]
+        shared = self._turn(d[:, None, q_rank + kv_rank:q_rank + kv_rank + rot_dim], pos, freqs, rot, magnitude, halves)[:, 0]
         page, off = self._physical(layer_cache.group, slots, pos)
         if bool((page < 0).any()):
             ctx.status |= 2
@@ -375,6 +386,76 @@ class EmulatedOps:
                     act = self.swiglu(gu) if alpha is None else self.gated_clamp(gu, alpha, limit)
                     out[r] += w * self.linear(act, w_down[e])[0].float()
         return out.to(h.dtype)
+
+    # ---- layer norms, the gated gelu, the delta rule with a decay per key channel ----------
+
+    @staticmethod
+    def _layernorm(x, w, b, eps):
+        xf = x.float()
+        c = xf - xf.mean(-1, keepdim=True)
+        return c * torch.rsqrt((c * c).mean(-1, keepdim=True) + eps) * w.float() + b.float()
+
+    def layernorm(self, x, delta, w, b, eps, out_dtype):
+        if delta is not None:
+            x.copy_((x.float() + delta.float()).to(x.dtype))
+        return self._layernorm(x, w, b, eps).to(out_dtype)
+
+    def embed_layernorm(self, tokens, table, w, b, eps, status):
+        return self._layernorm(self.embed(tokens, table, status), w, b, eps)
+
+    def gated_gelu(self, gu):
+        inter = gu.shape[1] // 2
+        g, u = gu[:, :inter].float(), gu[:, inter:].float()
+        return (torch.nn.functional.gelu(g, approximate="tanh") * u).to(gu.dtype)
+
+    def linear_gated_gelu(self, h, w_gate_up):
+        return self.gated_gelu(self.linear(h, w_gate_up))
+
+    def softcap(self, logits, cap):
+        return torch.tanh(logits / cap) * cap
+
+    def conv_unit_heads(self, ctx, p, weight, state, kv_heads, dim, q_scale, inner, n_inner, inner_width):
+        rows, taps = p.shape[0], weight.shape[1]
+        y = torch.zeros(p.shape, dtype=torch.float32, device=p.device)
+        for b in range(ctx.n_seqs):
+            slot, r0, r1 = int(ctx.seq_slot[b]), int(ctx.cu_q[b]), int(ctx.cu_q[b + 1])
+            past = state[slot].float() if taps > 1 else y.new_zeros((0, p.shape[1]))
+            hist = torch.cat([past, p[r0:r1].float()], dim=0)
+            for j in range(taps):
+                y[r0:r1] += weight[:, j].float()[None, :] * hist[j:j + (r1 - r0)]
+            if taps > 1:
+                state[slot] = hist[hist.shape[0] - (taps - 1):]
+        y = y * torch.sigmoid(y)
+        qk = y[:, :2 * kv_heads * dim].reshape(rows, 2, kv_heads, dim)
+        qk = qk * torch.rsqrt((qk * qk).sum(-1, keepdim=True) + 1e-6)
+        qk[:, 0] *= q_scale
+        y[:, :2 * kv_heads * dim] = qk.reshape(rows, -1)
+        low = torch.zeros((rows, inner_width), dtype=p.dtype, device=p.device)
+        low[:, :n_inner] = inner[:, :n_inner].to(p.dtype)
+        return y, low
+
+    def delta_scan(self, ctx, qkv, z, inner, b_col, a_log, dt_bias, norm, eps, state, heads, kv_heads, dim, vdim, out_dtype):
+        H, G, D, V = heads, kv_heads, dim, vdim
+        rows = qkv.shape[0]
+        q = qkv[:, :G * D].reshape(rows, G, D).repeat_interleave(H // G, dim=1)
+        k = qkv[:, G * D:2 * G * D].reshape(rows, G, D).repeat_interleave(H // G, dim=1)
+        v = qkv[:, 2 * G * D:].reshape(rows, H, V)
+        beta = torch.sigmoid(inner[:, b_col:b_col + H].float())
+        g = torch.exp(-torch.exp(a_log.float())[None, :, None]
+                      * torch.nn.functional.softplus(z[:, :H * D].float() + dt_bias.float(), threshold=80.0).reshape(rows, H, D))
+        out = torch.empty(rows, H, V, dtype=torch.float32, device=qkv.device)
+        cu = ctx.cu_q.tolist()
+        for b in range(ctx.n_seqs):
+            slot = int(ctx.seq_slot[b])
+            S = state[slot].reshape(H, D, V).clone()
+            for t in range(cu[b], cu[b + 1]):
+                S = g[t][:, :, None] * S
+                u = beta[t][:, None] * (v[t] - torch.einsum("hk,hkv->hv", k[t], S))
+                S = S + k[t][:, :, None] * u[:, None, :]
+                out[t] = torch.einsum("hk,hkv->hv", q[t], S)
+            state[slot] = S.reshape(-1)
+        o = out * torch.rsqrt((out * out).mean(-1, keepdim=True) + eps) * norm.float()
+        return (o.reshape(rows, H * V) * torch.sigmoid(z[:, H * D:].float())).to(out_dtype)
 
     def gather_rows(self, x, rows):
         return x[rows.long()].clone()
