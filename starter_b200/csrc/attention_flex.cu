@@ -146,11 +146,16 @@ __global__ void kv_store_kernel(const T* __restrict__ k, long long k_row, const 
     }
 }
 
-// Columns [0, rot) of every head turn in neighbouring pairs by position * freqs[pair]; later columns are copied.
-// angle, sine and cosine are 32-bit.
+// The two columns of pair c among the ``rot`` that turn: neighbours, or with ``halves`` rot / 2 apart.
+__device__ __forceinline__ int pair_first(int c, int halves) { return halves ? c : 2 * c; }
+__device__ __forceinline__ int pair_second(int c, int rot, int halves) { return halves ? c + rot / 2 : 2 * c + 1; }
+
+// Columns [0, rot) of every head turn in pairs by position * freqs[pair], sines and cosines times ``magnitude``; later
+// columns are copied.  angle, sine and cosine are 32-bit.
 template <class T>
 __global__ void rotate_pairs_kernel(const T* __restrict__ src, long long s_row, long long s_head, T* __restrict__ dst, long long d_row,
-                                    long long d_head, SbBatch batch, const float* __restrict__ freqs, int n_heads, int cols, int rot) {
+                                    long long d_head, SbBatch batch, const float* __restrict__ freqs, int n_heads, int cols, int rot,
+                                    float magnitude, int halves) {
     pdl_wait();
     const int row = blockIdx.x;
     int slot, pos;
@@ -163,28 +168,33 @@ __global__ void rotate_pairs_kernel(const T* __restrict__ src, long long s_row, 
         if (c < half) {
             float sn, cs;
             sincosf((float)pos * freqs[c], &sn, &cs);
-            const float a = to_f<T>(s[2 * c]), b = to_f<T>(s[2 * c + 1]);
-            d[2 * c] = from_f<T>(a * cs - b * sn);
-            d[2 * c + 1] = from_f<T>(b * cs + a * sn);
+            sn *= magnitude;
+            cs *= magnitude;
+            const int i = pair_first(c, halves), j = pair_second(c, rot, halves);
+            const float a = to_f<T>(s[i]), b = to_f<T>(s[j]);
+            d[i] = from_f<T>(a * cs - b * sn);
+            d[j] = from_f<T>(b * cs + a * sn);
         } else {
             d[rot + c - half] = s[rot + c - half];
         }
     }
 }
 
-// One block per row of down = [query latent (q_rank) | key/value latent (kv_rank) | shared rotated part (rot_dim)]:
-// the query latent normed into cq, the key/value latent normed and the shared part rotated into the row's one
-// cache row [kv_rank + rot_dim]; the same row also into row_out [rows, kv_rank + rot_dim] when that is given.
+// One block per row of down = [query latent (q_rank) | key/value latent (kv_rank) | shared rotated part (rot_dim) | more]
+// (rows ``ld`` elements apart): the query latent normed into cq, the key/value latent normed and the shared part rotated
+// into the row's one cache row [kv_rank + rot_dim]; the same row also into row_out [rows, kv_rank + rot_dim] when that is
+// given.  kv_rank 0: the query latent only (a layer that reads another layer's rows).
 template <class T, class W>
-__global__ void latent_prepare_kernel(const T* __restrict__ down, T* __restrict__ cq, SbBatch batch, SbFlex p, int q_rank, int kv_rank,
+__global__ void latent_prepare_kernel(const T* __restrict__ down, long long ld, T* __restrict__ cq, SbBatch batch, SbFlex p, int q_rank, int kv_rank,
                                       int rot_dim, const W* __restrict__ q_norm, const W* __restrict__ kv_norm, float eps,
-                                      const float* __restrict__ freqs, int rot, int* status, T* __restrict__ row_out) {
+                                      const float* __restrict__ freqs, int rot, float magnitude, int halves, int* status,
+                                      T* __restrict__ row_out) {
     __shared__ float red[33];
     pdl_wait();
     const int row = blockIdx.x;
     int slot, pos;
     row_place(batch, row, slot, pos);
-    const T* dr = down + (long long)row * (q_rank + kv_rank + rot_dim);
+    const T* dr = down + (long long)row * ld;
     T* ro = row_out != nullptr ? row_out + (long long)row * (kv_rank + rot_dim) : nullptr;
     float ss = 0.f;
     for (int c = threadIdx.x; c < q_rank; c += blockDim.x) {
@@ -195,6 +205,7 @@ __global__ void latent_prepare_kernel(const T* __restrict__ down, T* __restrict_
     float rstd = 1.0f / sqrtf(ss / (float)q_rank + eps);
     for (int c = threadIdx.x; c < q_rank; c += blockDim.x)
         cq[(long long)row * q_rank + c] = from_f<T>(__fmul_rn(__fmul_rn(to_f<T>(dr[c]), rstd), to_f<W>(q_norm[c])));
+    if (kv_rank == 0) return;
     const long long tok = flex_token(p, slot, pos, 0);
     ss = 0.f;
     for (int c = threadIdx.x; c < kv_rank; c += blockDim.x) {
@@ -219,13 +230,16 @@ __global__ void latent_prepare_kernel(const T* __restrict__ down, T* __restrict_
         if (c < half) {
             float sn, cs;
             sincosf((float)pos * freqs[c], &sn, &cs);
-            const float a = to_f<T>(sr[2 * c]), b = to_f<T>(sr[2 * c + 1]);
+            sn *= magnitude;
+            cs *= magnitude;
+            const int i = pair_first(c, halves), j = pair_second(c, rot, halves);
+            const float a = to_f<T>(sr[i]), b = to_f<T>(sr[j]);
             const T x = from_f<T>(a * cs - b * sn), y = from_f<T>(b * cs + a * sn);
-            kd[kv_rank + 2 * c] = x;
-            kd[kv_rank + 2 * c + 1] = y;
+            kd[kv_rank + i] = x;
+            kd[kv_rank + j] = y;
             if (ro != nullptr) {
-                ro[kv_rank + 2 * c] = x;
-                ro[kv_rank + 2 * c + 1] = y;
+                ro[kv_rank + i] = x;
+                ro[kv_rank + j] = y;
             }
         } else {
             kd[kv_rank + rot + c - half] = sr[rot + c - half];
@@ -263,27 +277,28 @@ int sb_kv_store(int dtype, const void* k, long long k_row, const void* v, long l
 }
 
 int sb_rotate_pairs(int dtype, const void* src, long long s_row, long long s_head, void* dst, long long d_row, long long d_head,
-                    SbBatch batch, const float* freqs, int n_heads, int cols, int rot, cudaStream_t stream) {
+                    SbBatch batch, const float* freqs, int n_heads, int cols, int rot, float magnitude, int halves, cudaStream_t stream) {
     if (batch.n_rows <= 0 || cols <= 0) return 0;
     if (rot < 0 || rot > cols || rot % 2) return (int)cudaErrorInvalidValue;
     if (dtype == SB_F32)
         sb_launch(rotate_pairs_kernel<float>, batch.n_rows, 128, 0, stream, (const float*)src, s_row, s_head, (float*)dst, d_row, d_head,
-                  batch, freqs, n_heads, cols, rot);
+                  batch, freqs, n_heads, cols, rot, magnitude, halves);
     else
         sb_launch(rotate_pairs_kernel<__nv_bfloat16>, batch.n_rows, 128, 0, stream, (const __nv_bfloat16*)src, s_row, s_head,
-                  (__nv_bfloat16*)dst, d_row, d_head, batch, freqs, n_heads, cols, rot);
+                  (__nv_bfloat16*)dst, d_row, d_head, batch, freqs, n_heads, cols, rot, magnitude, halves);
     SB_LAUNCH_CHECK();
 }
 
-int sb_latent_prepare(int dtype, int w_dtype, const void* down, void* cq, SbBatch batch, SbFlex p, int q_rank, int kv_rank, int rot_dim,
-                      const void* q_norm, const void* kv_norm, float eps, const float* freqs, int rot, int* status, void* row_out,
-                      cudaStream_t stream) {
+int sb_latent_prepare(int dtype, int w_dtype, const void* down, long long ld, void* cq, SbBatch batch, SbFlex p, int q_rank, int kv_rank,
+                      int rot_dim, const void* q_norm, const void* kv_norm, float eps, const float* freqs, int rot, float magnitude,
+                      int halves, int* status, void* row_out, cudaStream_t stream) {
     if (batch.n_rows <= 0) return 0;
-    if (rot < 0 || rot > rot_dim || rot % 2 || p.k_dim != kv_rank + rot_dim) return (int)cudaErrorInvalidValue;
+    if (rot < 0 || rot > rot_dim || rot % 2 || (kv_rank > 0 && p.k_dim != kv_rank + rot_dim) || ld < q_rank + kv_rank + rot_dim)
+        return (int)cudaErrorInvalidValue;
     typedef __nv_bfloat16 bf;
 #define SB_LP(T, W)                                                                                                          \
-    sb_launch(latent_prepare_kernel<T, W>, batch.n_rows, 128, 0, stream, (const T*)down, (T*)cq, batch, p, q_rank, kv_rank, rot_dim, \
-              (const W*)q_norm, (const W*)kv_norm, eps, freqs, rot, status, (T*)row_out)
+    sb_launch(latent_prepare_kernel<T, W>, batch.n_rows, 128, 0, stream, (const T*)down, ld, (T*)cq, batch, p, q_rank, kv_rank, \
+              rot_dim, (const W*)q_norm, (const W*)kv_norm, eps, freqs, rot, magnitude, halves, status, (T*)row_out)
     if (dtype == SB_F32 && w_dtype == SB_F32) SB_LP(float, float);
     else if (dtype == SB_BF16 && w_dtype == SB_BF16) SB_LP(bf, bf);
     else if (dtype == SB_BF16 && w_dtype == SB_F32) SB_LP(bf, float);

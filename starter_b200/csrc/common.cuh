@@ -62,6 +62,11 @@ __device__ __forceinline__ float xielu_value(float v, float a_pos, float a_neg) 
     return v > 0.f ? fmaf(a_pos * v, v, 0.5f * v) : fmaf(a_neg, expm1f(v) - v, 0.5f * v);
 }
 
+// The tanh form of gelu: z / 2 (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3))).
+__device__ __forceinline__ float gelu_tanh_value(float z) {
+    return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * fmaf(0.044715f * z * z, z, z)));
+}
+
 // Two 32-bit operations in one instruction (sm_100): a * b + c and a + b on pairs, each element rounded as the single
 // operation rounds it; and the largest of three.  For loops whose time is their instruction count.
 __device__ __forceinline__ float2 fma_pair(float2 a, float2 b, float2 c) {

@@ -4,7 +4,15 @@
 // be read out of, and written into, wider rows without a copy.  Each output is one running 32-bit sum over
 // k = 0..K-1 in order: a row's result does not depend on the rows around it.  It is the product of the 32-bit
 // path and of small shapes; many rows in bfloat16 go to the library's batched product.
+//
+// gate [rows, heads] (a view with a row stride; null: none): head h's outputs of row m are multiplied by
+// sigmoid(gate[m, h]), the product as it reads back from its type.  gate_heads is that step alone, for outputs that come
+// from elsewhere.
 #include "common.cuh"
+
+template <class T> __device__ __forceinline__ float head_sigmoid(const T* gate, long long gate_row, long long m, int head) {
+    return 1.0f / (1.0f + expf(-to_f<T>(gate[m * gate_row + head])));
+}
 
 #define GH_BM 64
 #define GH_BN 64
@@ -13,7 +21,7 @@
 template <class T>
 __global__ void __launch_bounds__(256) gemm_heads_kernel(const T* __restrict__ A, long long a_row, long long a_head,
                                                          const T* __restrict__ W, T* __restrict__ C, long long c_row,
-                                                         long long c_head, int M, int N, int K) {
+                                                         long long c_head, const T* __restrict__ gate, long long gate_row, int M, int N, int K) {
     __shared__ float As[GH_BK][GH_BM + 4];
     __shared__ float Ws[GH_BK][GH_BN + 4];
     pdl_wait();
@@ -56,10 +64,11 @@ __global__ void __launch_bounds__(256) gemm_heads_kernel(const T* __restrict__ A
     for (int i = 0; i < 4; ++i) {
         const int m = m0 + ty * 4 + i;
         if (m >= M) continue;
+        const float sig = gate != nullptr ? head_sigmoid<T>(gate, gate_row, m, head) : 1.0f;
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int n = n0 + tx * 4 + j;
-            if (n < N) Ch[m * c_row + n] = from_f<T>(acc[i][j]);
+            if (n < N) Ch[m * c_row + n] = from_f<T>(gate != nullptr ? rnd<T>(acc[i][j]) * sig : acc[i][j]);
         }
     }
 }
@@ -72,7 +81,7 @@ __global__ void __launch_bounds__(256) gemm_heads_kernel(const T* __restrict__ A
 template <class T>
 __global__ void __launch_bounds__(256) gemm_heads_rows_kernel(const T* __restrict__ A, long long a_row, long long a_head,
                                                               const T* __restrict__ W, T* __restrict__ C, long long c_row,
-                                                              long long c_head, int M, int N, int K) {
+                                                              long long c_head, const T* __restrict__ gate, long long gate_row, int M, int N, int K) {
     pdl_wait();
     const int head = blockIdx.y, lane = threadIdx.x & 31;
     const int n = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -92,32 +101,86 @@ __global__ void __launch_bounds__(256) gemm_heads_rows_kernel(const T* __restric
     for (int m = 0; m < GH_SMALL_M; ++m) {
         if (m < M) {
             const float v = warp_sum(acc[m]);
-            if (lane == 0) C[head * c_head + m * c_row + n] = from_f<T>(v);
+            if (lane == 0)
+                C[head * c_head + m * c_row + n] =
+                    from_f<T>(gate != nullptr ? rnd<T>(v) * head_sigmoid<T>(gate, gate_row, m, head) : v);
         }
     }
 }
 
+// out[m, h, :] = a[m, h, :] * sigmoid(gate[m, h]); a with a row and a head stride, out contiguous.  V8: eight bfloat16
+// columns at a time.
+template <class T, bool V8>
+__global__ void gate_heads_kernel(const T* __restrict__ a, long long a_row, long long a_head, const T* __restrict__ gate,
+                                  long long gate_row, T* __restrict__ out, long long rows, int H, int V) {
+    pdl_wait();
+    pdl_launch_dependents();
+    constexpr int W = V8 ? 8 : 1;
+    const long long n = rows * H * V / W;
+    for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
+        const long long mh = i * W / V, m = mh / H;
+        const int h = (int)(mh - m * H), c = (int)(i * W - mh * V);
+        const float sig = head_sigmoid<T>(gate, gate_row, m, h);
+        const T* src = a + m * a_row + h * a_head + c;
+        if (V8) {
+            const uint4 raw = *reinterpret_cast<const uint4*>(src);
+            const __nv_bfloat162* x = reinterpret_cast<const __nv_bfloat162*>(&raw);
+            uint4 res;
+            __nv_bfloat162* y = reinterpret_cast<__nv_bfloat162*>(&res);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const float2 f = __bfloat1622float2(x[e]);
+                y[e] = __floats2bfloat162_rn(f.x * sig, f.y * sig);
+            }
+            *reinterpret_cast<uint4*>(out + i * W) = res;
+        } else {
+            out[i] = from_f<T>(to_f<T>(*src) * sig);
+        }
+    }
+}
+
+extern "C" int sb_gate_heads(int dtype, const void* a, long long a_row, long long a_head, const void* gate, long long gate_row, void* out,
+                             int rows, int H, int V, cudaStream_t stream) {
+    if (rows <= 0 || H <= 0 || V <= 0) return 0;
+    typedef __nv_bfloat16 bf;
+    const long long n = (long long)rows * H * V;
+    const bool v8 = dtype == SB_BF16 && V % 8 == 0 && a_row % 8 == 0 && a_head % 8 == 0 && (reinterpret_cast<size_t>(a) & 15) == 0
+                    && (reinterpret_cast<size_t>(out) & 15) == 0;
+    const long long items = v8 ? n / 8 : n;
+    const int blocks = (int)((items + 255) / 256 < 8192 ? (items + 255) / 256 : 8192);
+    if (dtype == SB_F32)
+        sb_launch(gate_heads_kernel<float, false>, blocks, 256, 0, stream, (const float*)a, a_row, a_head, (const float*)gate, gate_row,
+                  (float*)out, (long long)rows, H, V);
+    else if (v8)
+        sb_launch(gate_heads_kernel<bf, true>, blocks, 256, 0, stream, (const bf*)a, a_row, a_head, (const bf*)gate, gate_row, (bf*)out,
+                  (long long)rows, H, V);
+    else
+        sb_launch(gate_heads_kernel<bf, false>, blocks, 256, 0, stream, (const bf*)a, a_row, a_head, (const bf*)gate, gate_row, (bf*)out,
+                  (long long)rows, H, V);
+    SB_LAUNCH_CHECK();
+}
+
 // Strides in elements.
 extern "C" int sb_gemm_heads(int dtype, const void* A, long long a_row, long long a_head, const void* W, void* C, long long c_row,
-                             long long c_head, int M, int N, int K, int heads, cudaStream_t stream) {
+                             long long c_head, const void* gate, long long gate_row, int M, int N, int K, int heads, cudaStream_t stream) {
     if (M <= 0 || N <= 0 || heads <= 0) return 0;
     if (M <= GH_SMALL_M && heads <= 65535) {
         dim3 small((N + 7) / 8, heads);
         if (dtype == SB_F32)
             sb_launch(gemm_heads_rows_kernel<float>, small, 256, 0, stream, (const float*)A, a_row, a_head, (const float*)W, (float*)C,
-                      c_row, c_head, M, N, K);
+                      c_row, c_head, (const float*)gate, gate_row, M, N, K);
         else
             sb_launch(gemm_heads_rows_kernel<__nv_bfloat16>, small, 256, 0, stream, (const __nv_bfloat16*)A, a_row, a_head,
-                      (const __nv_bfloat16*)W, (__nv_bfloat16*)C, c_row, c_head, M, N, K);
+                      (const __nv_bfloat16*)W, (__nv_bfloat16*)C, c_row, c_head, (const __nv_bfloat16*)gate, gate_row, M, N, K);
         SB_LAUNCH_CHECK();
     }
     dim3 grid((N + GH_BN - 1) / GH_BN, (M + GH_BM - 1) / GH_BM, heads);
     if (grid.y > 65535 || grid.z > 65535) return (int)cudaErrorInvalidValue;
     if (dtype == SB_F32)
         sb_launch(gemm_heads_kernel<float>, grid, 256, 0, stream, (const float*)A, a_row, a_head, (const float*)W, (float*)C, c_row,
-                  c_head, M, N, K);
+                  c_head, (const float*)gate, gate_row, M, N, K);
     else
         sb_launch(gemm_heads_kernel<__nv_bfloat16>, grid, 256, 0, stream, (const __nv_bfloat16*)A, a_row, a_head,
-                  (const __nv_bfloat16*)W, (__nv_bfloat16*)C, c_row, c_head, M, N, K);
+                  (const __nv_bfloat16*)W, (__nv_bfloat16*)C, c_row, c_head, (const __nv_bfloat16*)gate, gate_row, M, N, K);
     SB_LAUNCH_CHECK();
 }

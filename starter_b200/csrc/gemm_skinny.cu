@@ -50,6 +50,13 @@ int sb_gemm_skinny_gated(const void* A, const void* W, void* C, int M, int n_out
                                    SbSkinnyNorm{nullptr, 0.f, nullptr, 0, alpha, limit}, nullptr, partial, counters, stream);
 }
 
+// The same with gelu_tanh(g) * u, both halves as they read back from bfloat16.
+int sb_gemm_skinny_gelu(const void* A, const void* W, void* C, int M, int n_out, int K, int n_splits, int k_per_split, int tiled,
+                        int warps, float* partial, int* counters, cudaStream_t stream) {
+    return skinny_launch<false, 4>(A, W, C, M, n_out, K, n_splits, k_per_split, 1, 0, tiled, warps, 0,
+                                   SbSkinnyNorm{nullptr, 0.f, nullptr, 0, 0.f, 0.f, 0.f, 1}, nullptr, partial, counters, stream);
+}
+
 // A plain product with the two-sided activation in the epilogue: xielu(A W^T), a_pos z^2 + z / 2 for z > 0,
 // a_neg (exp(z) - 1 - z) + z / 2 otherwise, z the product as it reads back from bfloat16.
 int sb_gemm_skinny_xielu(const void* A, const void* W, void* C, int M, int n_out, int K, int n_splits, int k_per_split, int tiled,

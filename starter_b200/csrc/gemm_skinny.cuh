@@ -64,7 +64,9 @@ __device__ __forceinline__ float silu_mul_bf16(float g, float u) {
 }
 
 // gate and up as they read back from bfloat16 (what a product followed by an activation kernel would see), clamped.
-__device__ __forceinline__ float gated_act(float g, float u, float alpha, float limit) {
+// kind 1: the tanh form of gelu in silu's place.
+__device__ __forceinline__ float gated_act(float g, float u, float alpha, float limit, int kind) {
+    if (kind == 1) return gelu_tanh_value(__bfloat162float(__float2bfloat16_rn(g))) * __bfloat162float(__float2bfloat16_rn(u));
     if (limit > 0.f) {
         const float gb = fminf(__bfloat162float(__float2bfloat16_rn(g)), limit);
         const float ub = fminf(fmaxf(__bfloat162float(__float2bfloat16_rn(u)), -limit), limit);
@@ -93,6 +95,7 @@ struct SbSkinnyNorm {
     float act_limit;
     // what the epilogue of a plain product computes when act_unary is set, of the product as it reads back from
     // bfloat16: 1 the two-sided activation xielu_value(v, act_alpha, act_neg), 2 the squared relu max(v, 0)^2
+    // (with GATE_UP: 1 selects gelu_tanh(g) * u)
     float act_neg;
     int act_unary;
 };
@@ -312,7 +315,7 @@ gemm_skinny_kernel(const __nv_bfloat16* __restrict__ A, const __nv_bfloat16* __r
                     v += *cluster.map_shared_rank(&red[0][r][m], c);
                     if (GATE_UP) v2 += *cluster.map_shared_rank(&red[WPG][r][m], c);
                 }
-                if (GATE_UP) v = gated_act(v, v2, norm.act_alpha, norm.act_limit);
+                if (GATE_UP) v = gated_act(v, v2, norm.act_alpha, norm.act_limit, norm.act_unary);
                 else if (norm.act_unary) v = skinny_unary(__bfloat162float(__float2bfloat16_rn(v)), norm.act_unary, norm.act_alpha, norm.act_neg);
                 stored = skinny_store(C, (long long)m * n_out + n0 + r, v, out_f32, accumulate);
             }
@@ -347,7 +350,7 @@ gemm_skinny_kernel(const __nv_bfloat16* __restrict__ A, const __nv_bfloat16* __r
         float stored = 0.f;
         if (m < M && n0 + r < n_out) {
             float v = red[0][r][m];
-            if (GATE_UP) v = gated_act(v, red[WPG][r][m], norm.act_alpha, norm.act_limit);
+            if (GATE_UP) v = gated_act(v, red[WPG][r][m], norm.act_alpha, norm.act_limit, norm.act_unary);
             else if (norm.act_unary) v = skinny_unary(__bfloat162float(__float2bfloat16_rn(v)), norm.act_unary, norm.act_alpha, norm.act_neg);
             stored = skinny_store(C, (long long)m * n_out + n0 + r, v, out_f32, accumulate);
         }

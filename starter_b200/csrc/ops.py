@@ -52,6 +52,12 @@ class SbFlex(Structure):
                 ("pinned_pages", c_int), ("keep_first", c_int), ("softcap", c_float), ("talk", c_void_p)]
 
 
+class SbDelta(Structure):
+    _fields_ = [("qkv", c_void_p), ("z", c_void_p), ("z_ld", c_longlong), ("inner", c_void_p), ("inner_ld", c_longlong),
+                ("b_col", c_int), ("a_log", c_void_p), ("dt_bias", c_void_p), ("norm", c_void_p), ("eps", c_float),
+                ("state", c_void_p), ("state_slot", c_longlong), ("H", c_int), ("G", c_int), ("D", c_int), ("V", c_int)]
+
+
 def _code(dtype: torch.dtype) -> int:
     if dtype == torch.float32:
         return F32
@@ -113,16 +119,28 @@ class Ops:
                                    c_float, c_void_p],
             "sb_gated_clamp": [c_int, c_void_p, c_void_p, c_int, c_int, c_float, c_float, c_void_p],
             "sb_tanh": [c_int, c_void_p, c_void_p, c_longlong, c_void_p],
-            "sb_gemm_heads": [c_int, c_void_p, c_longlong, c_longlong, c_void_p, c_void_p, c_longlong, c_longlong, c_int, c_int,
-                              c_int, c_int, c_void_p],
+            "sb_gemm_heads": [c_int, c_void_p, c_longlong, c_longlong, c_void_p, c_void_p, c_longlong, c_longlong, c_void_p, c_longlong,
+                              c_int, c_int, c_int, c_int, c_void_p],
+            "sb_gate_heads": [c_int, c_void_p, c_longlong, c_longlong, c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_void_p],
             "sb_flex_attention_general": [c_int, SbFlex, SbBatch, c_void_p, c_void_p],
             "sb_flex_attention_mma": [SbFlex, SbBatch, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p],
             "sb_flex_attention_rows64": [SbFlex, SbBatch, c_void_p, c_int, c_int, c_void_p],
             "sb_kv_store": [c_int, c_void_p, c_longlong, c_void_p, c_longlong, SbBatch, SbFlex, c_int, c_float, c_void_p, c_void_p],
             "sb_rotate_pairs": [c_int, c_void_p, c_longlong, c_longlong, c_void_p, c_longlong, c_longlong, SbBatch, c_void_p,
-                                c_int, c_int, c_int, c_void_p],
-            "sb_latent_prepare": [c_int, c_int, c_void_p, c_void_p, SbBatch, SbFlex, c_int, c_int, c_int, c_void_p, c_void_p,
-                                  c_float, c_void_p, c_int, c_void_p, c_void_p, c_void_p],
+                                c_int, c_int, c_int, c_float, c_int, c_void_p],
+            "sb_latent_prepare": [c_int, c_int, c_void_p, c_longlong, c_void_p, SbBatch, SbFlex, c_int, c_int, c_int, c_void_p, c_void_p,
+                                  c_float, c_void_p, c_int, c_float, c_int, c_void_p, c_void_p, c_void_p],
+            "sb_layernorm": [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p],
+            "sb_embed_layernorm": [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p,
+                                   c_void_p],
+            "sb_gated_gelu": [c_int, c_void_p, c_void_p, c_int, c_int, c_void_p],
+            "sb_softcap": [c_void_p, c_longlong, c_float, c_void_p],
+            "sb_gemm_skinny_gelu": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
+                                    c_void_p],
+            "sb_conv_unit_heads": [c_int, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_longlong, SbBatch, c_int, c_int, c_int,
+                                   c_int, c_float, c_void_p, c_void_p, c_longlong, c_int, c_void_p, c_int, c_int, c_void_p],
+            "sb_delta_step": [c_int, SbDelta, SbBatch, c_void_p, c_void_p],
+            "sb_delta_chunk": [c_int, SbDelta, SbBatch, c_void_p, c_void_p, c_void_p, c_int, c_void_p],
             "sb_token_shift": [c_int, c_int, c_void_p, c_void_p, c_longlong, c_int, c_void_p, c_int, SbBatch, c_int, c_void_p,
                                c_void_p],
             "sb_wkv_scan": [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float,
@@ -176,6 +194,8 @@ class Ops:
         for fn in (lib.sb_flex_attention_mma_smem, lib.sb_flex_attention_rows64_smem, lib.sb_talking_attention_mma_smem):
             fn.argtypes = [c_int, c_int, c_int, c_int]
             fn.restype = c_longlong
+        lib.sb_delta_chunk_floats.argtypes = [c_int, c_int, c_int, c_int, c_int]
+        lib.sb_delta_chunk_floats.restype = c_longlong
         lib.sb_set_pdl.argtypes = [c_int]
         lib.sb_set_pdl.restype = None
         self._scratch = {}
@@ -482,7 +502,13 @@ class Ops:
         src = copy[0] if copy is not None else w
         tail = (M, n_out, K, n_splits, k_per_split, int(gate_up), int(out_float32), int(copy is not None), warps,
                 int(add_to is not None), _ptr(stats_out), _ptr(buf[0]), _ptr(buf[1]), self._stream())
-        if act is not None:   # (alpha, limit): the clamped activation in the epilogue of a [gate; up] product
+        if act == "gelu":   # gelu(gate) * up in the epilogue of a [gate; up] product
+            if not gate_up or norm is not None or add_to is not None or out_float32:
+                raise KernelError("the gated gelu sits in the epilogue of a plain [gate; up] product")
+            self._check(self.lib.sb_gemm_skinny_gelu(_ptr(a), _ptr(src), _ptr(out), M, n_out, K, n_splits, k_per_split,
+                                                     int(copy is not None), warps, _ptr(buf[0]), _ptr(buf[1]), self._stream()),
+                        "gemm_skinny_gelu")
+        elif act is not None:   # (alpha, limit): the clamped activation in the epilogue of a [gate; up] product
             if not gate_up or norm is not None or add_to is not None or out_float32:
                 raise KernelError("the clamped activation sits in the epilogue of a plain [gate; up] product")
             self._check(self.lib.sb_gemm_skinny_gated(_ptr(a), _ptr(src), _ptr(out), M, n_out, K, n_splits, k_per_split,
@@ -570,6 +596,59 @@ class Ops:
         if h.dtype == torch.bfloat16 and w_gate_up.dtype == torch.bfloat16 and K % 8 == 0 and M <= self.SKINNY_MAX_ROWS:
             return self._skinny(h, w_gate_up, w_gate_up.shape[0] // 2, True, False, act=(alpha, limit))
         return self.gated_clamp(self.linear(h, w_gate_up), alpha, limit)
+
+    def gated_gelu(self, gu):
+        """[g | u] -> gelu(g) * u with the tanh form of gelu."""
+        inter = gu.shape[1] // 2
+        if not gu.is_contiguous():
+            raise KernelError("gated_gelu: contiguous rows")
+        out = torch.empty((gu.shape[0], inter), dtype=gu.dtype, device=gu.device)
+        self._check(self.lib.sb_gated_gelu(_code(gu.dtype), _ptr(gu), _ptr(out), gu.shape[0], inter, self._stream()), "gated_gelu")
+        return out
+
+    def linear_gated_gelu(self, h, w_gate_up):
+        """gated_gelu(h @ w_gate_up^T) for a fused [gate; up] matrix.  For the few rows of a decode step the activation sits
+        in the product's epilogue, as SwiGLU does in ``linear_swiglu``."""
+        M, K = h.shape
+        if h.dtype == torch.bfloat16 and w_gate_up.dtype == torch.bfloat16 and K % 8 == 0 and M <= self.SKINNY_MAX_ROWS:
+            return self._skinny(h, w_gate_up, w_gate_up.shape[0] // 2, True, False, act="gelu")
+        return self.gated_gelu(self.linear(h, w_gate_up))
+
+    # ---- layer norms, the capped head ----------------------------------------------------
+
+    @staticmethod
+    def _norm_vectors(w, b, width, what):
+        for t in (w, b):
+            if t.dtype != torch.float32 or t.numel() != width or not t.is_contiguous():
+                raise KernelError(f"{what}: weight and bias are 32-bit, one number per column")
+
+    def layernorm(self, x, delta, w, b, eps, out_dtype):
+        """The layer norm of 32-bit rows x in ``out_dtype``; with ``delta`` (rows of that type) x += delta first, in place."""
+        if x.dtype != torch.float32 or not x.is_contiguous():
+            raise KernelError("layernorm: contiguous 32-bit rows")
+        if delta is not None and (delta.dtype != out_dtype or delta.shape != x.shape or not delta.is_contiguous()):
+            raise KernelError("layernorm: a branch output has the run's dtype and the residual's shape")
+        self._norm_vectors(w, b, x.shape[1], "layernorm")
+        out = torch.empty(x.shape, dtype=out_dtype, device=x.device)
+        self._check(self.lib.sb_layernorm(_code(out_dtype), _ptr(x), _ptr(delta), _ptr(w), _ptr(b), _ptr(out), x.shape[0], x.shape[1],
+                                          float(eps), self._stream()), "layernorm")
+        return out
+
+    def embed_layernorm(self, tokens, table, w, b, eps, status):
+        """The layer norm of the table's rows by token id, 32-bit."""
+        self._norm_vectors(w, b, table.shape[1], "embed_layernorm")
+        out = torch.empty((tokens.shape[0], table.shape[1]), dtype=torch.float32, device=table.device)
+        self._check(self.lib.sb_embed_layernorm(_code(table.dtype), _ptr(tokens), _ptr(table), _ptr(w), _ptr(b), _ptr(out),
+                                                tokens.shape[0], table.shape[1], table.shape[0], float(eps), _ptr(status),
+                                                self._stream()), "embed_layernorm")
+        return out
+
+    def softcap(self, logits, cap):
+        """cap * tanh(logits / cap), in place (32-bit)."""
+        if logits.dtype != torch.float32 or not logits.is_contiguous():
+            raise KernelError("softcap: contiguous 32-bit logits")
+        self._check(self.lib.sb_softcap(_ptr(logits), logits.numel(), float(cap), self._stream()), "softcap")
+        return logits
 
     # ---- attention ----------------------------------------------------------------------
 
@@ -783,20 +862,40 @@ class Ops:
 
     HEADS_LIBRARY_MIN_ROWS = 64
 
-    def linear_heads(self, a, w, out):
+    def gate_heads(self, a, gate):
+        """a [rows, heads, V] (a view, last axis contiguous) times sigmoid(gate [rows, heads], a view of wider rows), in a new
+        contiguous tensor."""
+        rows, H, V = a.shape
+        if a.stride(2) != 1 or tuple(gate.shape) != (rows, H) or gate.stride(1) != 1 or gate.dtype != a.dtype:
+            raise KernelError("gate_heads: one gate per row and head, in the run's dtype")
+        out = torch.empty((rows, H, V), dtype=a.dtype, device=a.device)
+        self._check(self.lib.sb_gate_heads(_code(a.dtype), _ptr(a), a.stride(0), a.stride(1), _ptr(gate), gate.stride(0), _ptr(out),
+                                           rows, H, V, self._stream()), "gate_heads")
+        return out
+
+    def linear_heads(self, a, w, out, gate=None):
         """out[m, h, :] = a[m, h, :] times w[h] transposed, for views a [rows, heads, K] and out [rows, heads, N] whose
-        last axis is contiguous (a head's columns inside wider rows) and w [heads, N, K]."""
+        last axis is contiguous (a head's columns inside wider rows) and w [heads, N, K].  ``gate`` [rows, heads] (a view of
+        wider rows; ``out`` is then contiguous): the product times sigmoid(gate), head by head."""
         rows, H, K = a.shape
         N = w.shape[1]
         if (tuple(w.shape) != (H, N, K) or tuple(out.shape) != (rows, H, N) or a.stride(2) != 1 or out.stride(2) != 1
                 or not w.is_contiguous() or not (a.dtype == w.dtype == out.dtype)):
             raise KernelError(f"linear_heads: a {tuple(a.shape)}, w {tuple(w.shape)}, out {tuple(out.shape)}")
+        if gate is not None and (tuple(gate.shape) != (rows, H) or gate.stride(1) != 1 or gate.dtype != a.dtype or not out.is_contiguous()):
+            raise KernelError("linear_heads: one gate per row and head, in the run's dtype")
         if a.dtype == torch.bfloat16 and rows > self.HEADS_LIBRARY_MIN_ROWS and K % 8 == 0 and N % 8 == 0:
             # many rows: the library's batched product on the tensor cores, as the plain products of a prompt
-            out.copy_(torch.bmm(a.transpose(0, 1), w.transpose(1, 2)).transpose(0, 1))
+            product = torch.bmm(a.transpose(0, 1), w.transpose(1, 2)).transpose(0, 1)
+            if gate is None:
+                out.copy_(product)
+            else:   # the gate's kernel puts the heads side by side as the copy would
+                self._check(self.lib.sb_gate_heads(_code(a.dtype), _ptr(product), product.stride(0), product.stride(1), _ptr(gate),
+                                                   gate.stride(0), _ptr(out), rows, H, N, self._stream()), "gate_heads")
             return out
         self._check(self.lib.sb_gemm_heads(_code(a.dtype), _ptr(a), a.stride(0), a.stride(1), _ptr(w), _ptr(out), out.stride(0),
-                                           out.stride(1), rows, N, K, H, self._stream()), "gemm_heads")
+                                           out.stride(1), _ptr(gate), gate.stride(0) if gate is not None else 0, rows, N, K, H,
+                                           self._stream()), "gemm_heads")
         return out
 
     def _flex(self, layer_cache, q=None, n_heads=0, scale=1.0, v_dim=None, values_in_keys=False, sink=None, head_scale=None,
@@ -914,9 +1013,10 @@ class Ops:
                                          int(value_norm_eps is not None), float(value_norm_eps or 0.0), _ptr(ctx.status),
                                          self._stream()), "kv_store")
 
-    def rotate_pairs(self, ctx, src, dst, freqs, rot):
+    def rotate_pairs(self, ctx, src, dst, freqs, rot, magnitude=1.0, halves=False):
         """dst = src [rows, heads, cols] (views, last axis contiguous) with the first ``rot`` columns of every head
-        turned in neighbouring pairs by the row's position times ``freqs`` (32-bit, [rot / 2])."""
+        turned in neighbouring pairs (with ``halves``: column i with column i + rot / 2) by the row's position times
+        ``freqs`` (32-bit, [rot / 2]), sines and cosines times ``magnitude``."""
         rows, H, cols = src.shape
         if tuple(dst.shape) != (rows, H, cols) or src.stride(2) != 1 or dst.stride(2) != 1 or src.dtype != dst.dtype:
             raise KernelError("rotate_pairs: source and destination differ")
@@ -925,25 +1025,31 @@ class Ops:
         elif freqs.dtype != torch.float32 or freqs.numel() * 2 != rot:
             raise KernelError("rotate_pairs: one 32-bit frequency per pair")
         self._check(self.lib.sb_rotate_pairs(_code(src.dtype), _ptr(src), src.stride(0), src.stride(1), _ptr(dst), dst.stride(0),
-                                             dst.stride(1), self._batch(ctx), _ptr(freqs), H, cols, int(rot), self._stream()),
-                    "rotate_pairs")
+                                             dst.stride(1), self._batch(ctx), _ptr(freqs), H, cols, int(rot), float(magnitude),
+                                             int(bool(halves)), self._stream()), "rotate_pairs")
 
-    def latent_prepare(self, ctx, down, layer_cache, q_rank, kv_rank, rot_dim, q_norm, kv_norm, eps, freqs, rot, rows_too=False):
-        """down [rows, q_rank + kv_rank + rot_dim] -> the normed query latent [rows, q_rank]; the normed key/value
-        latent and the rotated shared part go to the row's place in the layer's cache.  ``rows_too``: what went to the
-        cache is returned as well, (cq, [rows, kv_rank + rot_dim])."""
-        if down.shape[1] != q_rank + kv_rank + rot_dim or not down.is_contiguous() or q_norm.dtype != kv_norm.dtype:
+    def latent_prepare(self, ctx, down, layer_cache, q_rank, kv_rank, rot_dim, q_norm, kv_norm, eps, freqs=None, rot=0, magnitude=1.0,
+                       halves=False, rows_too=False):
+        """down [rows, q_rank + kv_rank + rot_dim, possibly more] -> the normed query latent [rows, q_rank]; the normed
+        key/value latent and the rotated shared part (turned as ``rotate_pairs`` does) go to the row's place in the layer's
+        cache.  ``rows_too``: what went to the cache is returned as well, (cq, [rows, kv_rank + rot_dim]).  ``layer_cache``
+        None: the query latent only."""
+        store = layer_cache is not None
+        if not store:
+            kv_rank = rot_dim = 0
+        if down.shape[1] < q_rank + kv_rank + rot_dim or down.stride(1) != 1 or (store and q_norm.dtype != kv_norm.dtype):
             raise KernelError("latent_prepare: the down-projection has the wrong width")
         if down.dtype == torch.float32 and q_norm.dtype != torch.float32:
             raise KernelError("a float32 run needs float32 norm weights")
-        if freqs is None:
-            rot = 0
-        p = self._flex(layer_cache, values_in_keys=True)
+        if freqs is None or not store:
+            freqs, rot = None, 0
+        p = self._flex(layer_cache, values_in_keys=True) if store else SbFlex()
         cq = torch.empty((down.shape[0], q_rank), dtype=down.dtype, device=down.device)
         kept = torch.empty((down.shape[0], kv_rank + rot_dim), dtype=down.dtype, device=down.device) if rows_too else None
-        self._check(self.lib.sb_latent_prepare(_code(down.dtype), _code(q_norm.dtype), _ptr(down), _ptr(cq), self._batch(ctx), p,
-                                               q_rank, kv_rank, rot_dim, _ptr(q_norm), _ptr(kv_norm), float(eps), _ptr(freqs),
-                                               int(rot), _ptr(ctx.status), _ptr(kept), self._stream()), "latent_prepare")
+        self._check(self.lib.sb_latent_prepare(_code(down.dtype), _code(q_norm.dtype), _ptr(down), down.stride(0), _ptr(cq),
+                                               self._batch(ctx), p, q_rank, kv_rank, rot_dim, _ptr(q_norm), _ptr(kv_norm), float(eps),
+                                               _ptr(freqs), int(rot), float(magnitude), int(bool(halves)), _ptr(ctx.status), _ptr(kept),
+                                               self._stream()), "latent_prepare")
         return (cq, kept) if rows_too else cq
 
     def token_shift(self, ctx, h, state, prev_offset, mu):
@@ -1207,6 +1313,69 @@ class Ops:
         if raw is not None:
             self.launches += 1   # the norm and the gate
         return y
+
+    # ---- the delta rule with a decay per key channel ---------------------------------------
+
+    def conv_unit_heads(self, ctx, p, weight, state, kv_heads, dim, q_scale, inner, n_inner, inner_width):
+        """p [rows, channels] = [q heads | k heads | v], ``kv_heads`` heads of ``dim`` for q and k: a short causal convolution
+        per channel (``weight`` [channels, taps], 32-bit; ``state`` [slots, taps - 1, channels] holds each sequence's last
+        inputs and is brought up to date), silu, and for q and k the unit length per head (q times ``q_scale``); 32-bit
+        rows.  Beside them [rows, inner_width] in p's type: the first ``n_inner`` columns of ``inner`` (32-bit), then zeros.
+        The value heads' number does not matter here: their channels are dealt out 128 at a time."""
+        rows, C = p.shape
+        taps = weight.shape[1]
+        V = C - 2 * kv_heads * dim
+        if (p.stride(1) != 1 or tuple(weight.shape) != (C, taps) or weight.dtype != torch.float32 or not weight.is_contiguous() or V < 1
+                or inner.dtype != torch.float32 or inner.shape[0] != rows or inner.stride(1) != 1 or inner.shape[1] < n_inner):
+            raise KernelError("conv_unit_heads: rows of queries, keys and values, 32-bit [channels, taps] weights and inner vectors")
+        if taps > 1 and (state is None or state.dtype != torch.float32 or tuple(state.shape[1:]) != (taps - 1, C) or not state.is_contiguous()):
+            raise KernelError(f"conv_unit_heads: the state is [slots, {taps - 1}, {C}] 32-bit numbers")
+        piece = next((n for n in (128, 96, 64, 32) if V % n == 0), V)
+        out = torch.empty((rows, C), dtype=torch.float32, device=p.device)
+        low = torch.empty((rows, inner_width), dtype=p.dtype, device=p.device)
+        one_row = ctx.max_q_len == 1
+        self._check(self.lib.sb_conv_unit_heads(_code(p.dtype), _ptr(p), p.stride(0), _ptr(weight), taps,
+                                                _ptr(state) if taps > 1 else None, state.stride(0) if taps > 1 else 0, self._batch(ctx),
+                                                kv_heads, dim, V // piece, piece, float(q_scale), _ptr(out), _ptr(inner), inner.stride(0),
+                                                int(n_inner), _ptr(low), int(inner_width), int(one_row), self._stream()), "conv_unit_heads")
+        if taps > 1 and not one_row:
+            self.launches += 1   # the record's kernel
+        return out, low
+
+    DELTA_CHUNK_MIN_ROWS = 12   # a step whose longest sequence brings fewer rows walks them token by token
+
+    def delta_scan(self, ctx, qkv, z, inner, b_col, a_log, dt_bias, norm, eps, state, heads, kv_heads, dim, vdim, out_dtype):
+        """The gated delta rule over every sequence's rows, from and back into ``state`` [slots, heads * dim * vdim]: qkv
+        [rows, 2 kv_heads * dim + heads * vdim] (unit queries and keys, values), z [rows, heads * (dim + vdim)] (the decays'
+        inputs, then the gates'), inner[:, b_col + h] the step sizes before their sigmoid; all 32-bit.  Returns
+        RMSNorm_head(o) * norm * sigmoid(gate), [rows, heads * vdim] in ``out_dtype``.  Steps of a few rows per sequence walk
+        them token by token, longer ones sixteen at a time."""
+        rows = qkv.shape[0]
+        H, G, D, V = heads, kv_heads, dim, vdim
+        for t in (qkv, z, inner, a_log, dt_bias, norm, state):
+            if t.dtype != torch.float32 or t.stride(-1) != 1:
+                raise KernelError("delta_scan: everything that enters the recurrence is 32-bit")
+        if (qkv.shape[1] != 2 * G * D + H * V or not qkv.is_contiguous() or tuple(z.shape) != (rows, H * (D + V)) or inner.shape[0] != rows
+                or inner.shape[1] < b_col + H or a_log.numel() != H or dt_bias.numel() != H * D or norm.numel() != V
+                or state.shape[1] != H * D * V):
+            raise KernelError("delta_scan: sizes do not fit")
+        p = SbDelta(_ptr(qkv), _ptr(z), z.stride(0), _ptr(inner), inner.stride(0), int(b_col), _ptr(a_log), _ptr(dt_bias), _ptr(norm),
+                    float(eps), _ptr(state), state.stride(0), H, G, D, V)
+        y = torch.empty((rows, H * V), dtype=out_dtype, device=qkv.device)
+        floats = self.lib.sb_delta_chunk_floats(rows, ctx.n_seqs, H, D, V) if ctx.max_q_len >= self.DELTA_CHUNK_MIN_ROWS else -1
+        if floats < 0:
+            self._check(self.lib.sb_delta_step(_code(out_dtype), p, self._batch(ctx), _ptr(y), self._stream()), "delta_step")
+            return y
+        ws = torch.empty(floats, dtype=torch.float32, device=qkv.device)
+        raw = torch.empty((rows, H * V), dtype=torch.float32, device=qkv.device)
+        self._check(self.lib.sb_delta_chunk(_code(out_dtype), p, self._batch(ctx), _ptr(ws), _ptr(raw), _ptr(y),
+                                            self.delta_columns(ctx.n_seqs, H, V), self._stream()), "delta_chunk")
+        self.launches += 2   # the chunks' preparation, the walk, the norm and the gate
+        return y
+
+    def delta_columns(self, n_seqs: int, heads: int, vdim: int) -> int:
+        """Value columns per block of the walk over chunks: 16, or 8 while that leaves SMs without a block."""
+        return 16 if n_seqs * heads * -(-vdim // 16) >= self.sm_count() else 8
 
     def moe_route(self, h, router, correction, top, scale, bias=None, over_chosen=False):
         """(chosen int32 [rows, top], weight 32-bit [rows, top]) of softmax(h router^T + bias) (32-bit): the ``top`` largest
