@@ -491,8 +491,35 @@ PADITAR_SIZES = {
     "2048": (_paditar_raw(2048, dict(heads=8, kv_heads=4, dim=128, vdim=128), dict(heads=8, kv_heads=4, dim=128),
                           dict(heads=16, dim=64, vdim=128), ff=8192), NAZULORN_SIZES["2048"][0]),
 }
+
+
+def _siparax_raw(width, latent, delta, ff, vocab=32000):
+    """A Siparax configuration of six layers: the delta rule, gated latent attention, latent attention, twice, the second
+    gated one over the first one's latents."""
+    def layer(kind, extra=()):
+        mixer = dict(latent, scale=(latent["dim"] + latent["rot_dim"]) ** -0.5,
+                     rot={"base": 500000.0, "dims": latent["rot_dim"],
+                          "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}, **dict(extra))
+        return {"type": kind, "mixer": mixer}
+    recurrent = {"type": "channel_delta", "mixer": dict(delta, conv=4)}
+    kinds = [recurrent, layer("latent_attention_2"), layer("latent_attention"),
+             recurrent, layer("latent_attention_2", {"kv_from": 1}), layer("latent_attention")]
+    return {"architecture": "Siparax", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "logit_softcap": 30.0,
+            "layers": [dict(kind, mlp={"kind": "dense", "ff": ff}) for kind in kinds]}
+
+
+# Siparax beside Kudazen (the closest design the library has: attention through latents, a recurrence with a matrix state
+# and a data-dependent decay per key channel, a gated dense feed-forward, a 32-bit residual) at the same width, layers,
+# vocabulary and feed-forward; the latent attention and the recurrence have Kudazen's head counts and sizes.
+SIPARAX_SIZES = {
+    "1024": (_siparax_raw(1024, dict(heads=8, dim=64, rot_dim=32, vdim=64, q_rank=384, kv_rank=256),
+                          dict(heads=16, kv_heads=16, dim=64, vdim=64, decay_rank=64, gate_rank=64), ff=4096), FAMILY_SIZES["1024"][0]),
+    "2048": (_siparax_raw(2048, dict(heads=16, dim=128, rot_dim=64, vdim=128, q_rank=768, kv_rank=512),
+                          dict(heads=32, kv_heads=32, dim=64, vdim=64, decay_rank=64, gate_rank=64), ff=8192), FAMILY_SIZES["2048"][0]),
+}
 FAMILIES = {"kudazen": (FAMILY_SIZES, "qwen3", "Qwen3ForCausalLM"), "nazulorn": (NAZULORN_SIZES, "kudazen", "Kudazen"),
-            "gulazen": (GULAZEN_SIZES, "nazulorn", "Nazulorn"), "paditar": (PADITAR_SIZES, "nazulorn", "Nazulorn")}
+            "gulazen": (GULAZEN_SIZES, "nazulorn", "Nazulorn"), "paditar": (PADITAR_SIZES, "nazulorn", "Nazulorn"),
+            "siparax": (SIPARAX_SIZES, "kudazen", "Kudazen")}
 
 
 class TimedOps:
@@ -517,7 +544,7 @@ class TimedOps:
     def _cost(self, name, args, kwargs, out):
         nbytes = self._nbytes(args) + self._nbytes(kwargs.values()) + self._nbytes([out])
         flops = 0.0
-        if name in ("linear", "linear_swiglu", "linear_xielu", "linear_relu2", "linear_bias"):
+        if name in ("linear", "linear_swiglu", "linear_xielu", "linear_relu2", "linear_bias", "linear_gated_clamp", "linear_gated_gelu"):
             a, w = args[0], args[1]
             flops = 2.0 * a.shape[0] * w.shape[0] * w.shape[1]
         elif name == "linear_heads":
@@ -556,6 +583,16 @@ class TimedOps:
             q, heads, dim, vdim = args[1], args[12], args[13], args[14]
             flops = 6.0 * q.shape[0] * heads * dim * vdim
             nbytes = 2 * args[0].n_seqs * heads * dim * vdim * 4 + q.shape[0] * heads * (2 * dim * 2 + 3 * vdim * 2 + dim * 4)
+        elif name == "delta_scan":
+            qkv, z, heads, dim, vdim = args[1], args[2], args[10], args[12], args[13]
+            flops = 7.0 * qkv.shape[0] * heads * dim * vdim       # decay, what the key holds, the write, the read
+            nbytes = 2 * args[0].n_seqs * heads * dim * vdim * 4 + (qkv.numel() + z.numel() + qkv.shape[0] * heads) * 4 + self._nbytes([out])
+        elif name == "conv_unit_heads":
+            p, weight, inner = args[1], args[2], args[7]
+            nbytes = self._nbytes([p, weight, inner, out])
+        elif name == "layernorm":
+            x, delta = args[0], args[1]
+            nbytes = self._nbytes([x, x, delta, out] if delta is not None else [x, out])
         elif name == "mlstm_scan":
             q, heads, dim, vdim = args[1], args[15], args[16], args[17]
             flops = 6.0 * q.shape[0] * heads * dim * (vdim + 1)
@@ -598,7 +635,8 @@ class TimedOps:
                     req = args[2].group.request
                     label += ("[latent]" if kwargs.get("values_in_keys") else
                               "[keys as values]" if kwargs.get("sink") is not None and req.v_dim == req.head_dim and args[2].aux is not None else
-                              "[latent, narrow form]" if kwargs.get("sink") is not None else
+                              "[latent, narrow form]" if kwargs.get("sink") is not None or "slopes" not in kwargs and
+                              args[2].group.v_heads == args[2].group.request.num_kv_heads else
                               "[two maps]" if args[2].group.v_heads != args[2].group.request.num_kv_heads else "[chunked]")
                 self.records.append((label, t0, t1) + self._cost(name, args, kwargs, out))
             return out
@@ -679,9 +717,9 @@ def _family_arm(torch, raw, peaks, prefill_tokens, batch, context, steps, warmup
 
 
 def run_family(args) -> int:
-    """--family kudazen | nazulorn | gulazen | paditar: the design at a few sizes that resemble a real model's layers (random weights),
+    """--family kudazen | nazulorn | gulazen | paditar | siparax: the design at a few sizes that resemble a real model's layers (random weights),
     beside the library's closest model of the same width, feed-forward work per token, layer count and vocabulary (Kudazen
-    beside the Qwen3 decoder, Nazulorn beside Kudazen, Gulazen and Paditar beside Nazulorn).  One JSON line."""
+    beside the Qwen3 decoder, Nazulorn and Siparax beside Kudazen, Gulazen and Paditar beside Nazulorn).  One JSON line."""
     import torch
     peaks, peak_source = load_peaks()
     torch.cuda.set_device(0)
@@ -909,10 +947,10 @@ def main() -> int:
     ap.add_argument("--context", type=int, default=0)
     ap.add_argument("--skip-points", action="store_true", help="leave out the further decode points")
     ap.add_argument("--skip-e2e", action="store_true")
-    ap.add_argument("--family", default="", choices=["", "kudazen", "nazulorn", "gulazen", "paditar"],
+    ap.add_argument("--family", default="", choices=["", "kudazen", "nazulorn", "gulazen", "paditar", "siparax"],
                     help="instead of the default workload: this model family at a few layer sizes, beside the library's closest "
-                         "model of equal size (kudazen beside the Qwen3 shape, nazulorn beside kudazen, gulazen and paditar beside "
-                         "nazulorn)")
+                         "model of equal size (kudazen beside the Qwen3 shape, nazulorn and siparax beside kudazen, gulazen and paditar "
+                         "beside nazulorn)")
     ap.add_argument("--sizes", default="", help="with --family: sizes to run, with commas between them (default: all)")
     args = ap.parse_args()
 

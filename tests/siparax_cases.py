@@ -1,7 +1,7 @@
 """Small Siparax configurations for the tests, and the plain implementation's logits for them.
 
 The configurations differ from one another in every size and option: 1, 2, 3, 5 and 8 taps; as many query/key heads as
-value heads, fewer, and one; key and value sizes that differ either way, sizes of one column, beyond the 128 key
+value heads, fewer, and one; key and value sizes that differ either way, sizes of two columns, beyond the 128 key
 channels and 128 value columns that registers hold, and no multiples of 4 or 8; inner sizes of the decay and of the gate
 that differ; latents of widths the tensor-core kernels take and do not; one head; rotations stretched (with ramps inside,
 above and below the pairs) and plain; rotated parts of 2 columns and more; layers that read another layer's latents, next
@@ -85,11 +85,11 @@ CASES = {
         _with(_halves(1, 16, 6, 12, 8, 16, 300.0, (3.0, 100, 10.0, 0.5), kv_from=1), None),
         _with(_delta(8, 4, 8, 136, 2, 8, 16), 48)]),
     # a width that is no multiple of 4, odd sizes everywhere (rows that no 16-byte read fits), an odd vocabulary, eight taps,
-    # heads of one column
+    # keys of two columns
     "E": _model(131, 30, 1e-6, 20.0, [
         _with(_delta(3, 1, 7, 5, 8, 3, 9), 14),
         _with(_pairs(7, 5, 6, 3, 11, 13, 700.0, STRETCH), 22),
-        _with(_delta(5, 5, 1, 1, 2, 1, 1), None),
+        _with(_delta(5, 5, 2, 3, 2, 1, 1), None),
         _with(_halves(5, 3, 2, 7, 9, 65, 40.0, (2.0, 20, 2.0, 1.0)), 10)]),
 }
 SEEDS = {"A": 45, "B": 46, "C": 47, "D": 48, "E": 49}
