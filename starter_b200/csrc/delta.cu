@@ -12,66 +12,117 @@
 // Convolution, silu, unit norms, decays, state, sums, the output's norm and gate are 32-bit in every run.
 #include "delta.cuh"
 
-// A warp per (row, head of q, k or v).  p [rows, C] in the run's type, rows ld apart, C = 2 G D + H V channels; record of a
-// sequence [taps - 1][C] floats.  inner [rows, inner_ld] 32-bit: its first n_inner columns are rounded into low [rows,
-// low_ld], zeros beyond.  ADVANCE (a step of one row per sequence): the thread that owns a channel also moves its record on.
-template <class T, bool ADVANCE>
+// A warp per (R consecutive rows, head of q, k or v), so that the loads of R rows are in flight together.  p [rows, C] in the
+// run's type, rows ld apart, C = 2 G D + H V channels; w [taps][C]; record of a sequence [taps - 1][C] floats.  inner [rows,
+// inner_ld] 32-bit: its first n_inner columns are rounded into low [rows, low_ld], zeros beyond.  ADVANCE (a step of one row
+// per sequence, R 1): the thread that owns a channel also moves its record on.  TAPS (0: any number): the number of taps
+// when rows that have all their inputs within the step are to be taken R at a time, each input read once.
+template <class T, int R, bool ADVANCE, int TAPS>
 __global__ void conv_unit_heads_kernel(const T* __restrict__ p, long long ld, const float* __restrict__ w, int taps, float* state,
                                        long long state_slot, SbBatch batch, int G, int D, int H, int V, float q_scale,
                                        float* __restrict__ out, const float* __restrict__ inner, long long inner_ld, int n_inner,
                                        T* __restrict__ low, int low_ld) {
     pdl_wait();
     const int lane = threadIdx.x & 31;
-    const long long wid = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-    const int units = 2 * G + H + 1;
-    const long long row = wid / units;
-    const int unit = (int)(wid - row * units);
-    if (row >= batch.n_rows) return;
-    if (unit == 2 * G + H) {   // the row's inner vectors, side by side in the run's type
-        for (int c = lane; c < low_ld; c += 32)
-            low[row * low_ld + c] = from_f<T>(c < n_inner ? inner[row * inner_ld + c] : 0.f);
+    const unsigned int wid = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    const unsigned int units = 2 * G + H + 1;
+    const int unit = (int)(wid % units);
+    const int r0 = (int)(wid / units) * R, n_here = min(R, batch.n_rows - r0);
+    if (n_here <= 0) return;
+    if (unit == 2 * G + H) {   // the rows' inner vectors, side by side in the run's type
+        for (int r = 0; r < n_here; ++r)
+            for (int c = lane; c < low_ld; c += 32)
+                low[(long long)(r0 + r) * low_ld + c] = from_f<T>(c < n_inner ? inner[(r0 + r) * inner_ld + c] : 0.f);
         return;
     }
-    const int s = batch.row_seq[row], first = batch.cu_q[s], keep = taps - 1;
-    const int t = (int)row - first;
+    const int keep = taps - 1;
     const bool is_v = unit >= 2 * G;
     const int size = is_v ? V : D, c0 = is_v ? 2 * G * D + (unit - 2 * G) * V : unit * D;
     const int C = 2 * G * D + H * V;
-    float* rec = keep > 0 ? state + (long long)batch.seq_slot[s] * state_slot : nullptr;
-    const T* seq = p + (long long)first * ld;
-    float* dst = out + row * C + c0;
-    float kept[DS_KEEP];   // a lane's values of a head of up to 32 * DS_KEEP columns; wider heads are read back from `dst`
-    float ss = 0.f;
-    auto value = [&](int c) {
+    int ahead[R];              // rows of its sequence that the step holds before row r
+    float* rec[R];
+#pragma unroll
+    for (int r = 0; r < R; ++r) {
+        const int row = r0 + min(r, n_here - 1), s = batch.row_seq[row];
+        ahead[r] = row - batch.cu_q[s];
+        rec[r] = keep > 0 ? state + (long long)batch.seq_slot[s] * state_slot : nullptr;
+    }
+    // all R rows are rows of one sequence with every input among the step's rows
+    const bool inside = TAPS > 0 && n_here == R && ahead[0] >= TAPS - 1 && ahead[R - 1] == ahead[0] + R - 1;
+    float kept[R][DS_KEEP], ss[R];   // a lane's values of a head of up to 32 * DS_KEEP columns; wider heads are read back from `out`
+    auto values = [&](int c, float (&y)[R]) {
         const int ch = c0 + c;
-        float y = 0.f;
+#pragma unroll
+        for (int r = 0; r < R; ++r) y[r] = 0.f;
+        if (TAPS > 0 && inside) {
+            constexpr int N = TAPS > 0 ? TAPS : 1;
+            const T* src = p + (long long)(r0 - (N - 1)) * ld + ch;
+            float wj[N], u[R + N - 1];
+#pragma unroll
+            for (int j = 0; j < N; ++j) wj[j] = w[(long long)j * C + ch];
+#pragma unroll
+            for (int m = 0; m < R + N - 1; ++m) {
+                u[m] = to_f<T>(*src);
+                src += ld;
+            }
+#pragma unroll
+            for (int r = 0; r < R; ++r)
+#pragma unroll
+                for (int j = 0; j < N; ++j) y[r] = fmaf(wj[j], u[r + j], y[r]);
+        } else
+#pragma unroll 4
         for (int j = 0; j < taps; ++j) {
-            const int src = t - keep + j;
-            const float u = src >= 0 ? to_f<T>(seq[(long long)src * ld + ch]) : rec[(long long)(keep + src) * C + ch];
-            y = fmaf(w[(long long)ch * taps + j], u, y);
-            if (ADVANCE && j > 0) rec[(long long)(j - 1) * C + ch] = u;   // entry j - 1 was read in an earlier turn
+            const float wj = w[(long long)j * C + ch];
+#pragma unroll
+            for (int r = 0; r < R; ++r) {
+                const int row = r0 + min(r, n_here - 1), back = keep - j;
+                const float u = ahead[r] >= back ? to_f<T>(p[(long long)(row - back) * ld + ch]) : rec[r][(long long)(ahead[r] + j) * C + ch];
+                y[r] = fmaf(wj, u, y[r]);
+                if (ADVANCE && j > 0) rec[r][(long long)(j - 1) * C + ch] = u;   // entry j - 1 was read in an earlier turn
+            }
         }
-        return y / (1.0f + expf(-y));
+#pragma unroll
+        for (int r = 0; r < R; ++r) y[r] = __fdividef(y[r], 1.0f + expf(-y[r]));
     };
 #pragma unroll
-    for (int i = 0; i < DS_KEEP; ++i) {
-        const int c = i * 32 + lane;
-        kept[i] = c < size ? value(c) : 0.f;
-        ss = fmaf(kept[i], kept[i], ss);
-    }
-    for (int c = DS_KEEP * 32 + lane; c < size; c += 32) {
-        const float y = value(c);
-        dst[c] = y;
-        ss = fmaf(y, y, ss);
-    }
-    float mul = 1.0f;
-    if (!is_v) mul = (unit < G ? q_scale : 1.0f) / sqrtf(warp_sum(ss) + 1e-6f);
+    for (int r = 0; r < R; ++r) ss[r] = 0.f;
 #pragma unroll
     for (int i = 0; i < DS_KEEP; ++i) {
-        const int c = i * 32 + lane;
-        if (c < size) dst[c] = kept[i] * mul;
+        float y[R];
+        if (i * 32 + lane < size) {
+            values(i * 32 + lane, y);
+        } else {
+#pragma unroll
+            for (int r = 0; r < R; ++r) y[r] = 0.f;
+        }
+#pragma unroll
+        for (int r = 0; r < R; ++r) {
+            kept[r][i] = y[r];
+            ss[r] = fmaf(y[r], y[r], ss[r]);
+        }
     }
-    for (int c = DS_KEEP * 32 + lane; c < size; c += 32) dst[c] *= mul;
+    for (int c = DS_KEEP * 32 + lane; c < size; c += 32) {
+        float y[R];
+        values(c, y);
+#pragma unroll
+        for (int r = 0; r < R; ++r) {
+            if (r < n_here) out[(long long)(r0 + r) * C + c0 + c] = y[r];
+            ss[r] = fmaf(y[r], y[r], ss[r]);
+        }
+    }
+    const float top = unit < G ? q_scale : 1.0f;
+#pragma unroll
+    for (int r = 0; r < R; ++r) {
+        if (r >= n_here) break;
+        const float mul = is_v ? 1.0f : top / sqrtf(warp_sum(ss[r]) + 1e-6f);
+        float* dst = out + (long long)(r0 + r) * C + c0;
+#pragma unroll
+        for (int i = 0; i < DS_KEEP; ++i) {
+            const int c = i * 32 + lane;
+            if (c < size) dst[c] = kept[r][i] * mul;
+        }
+        for (int c = DS_KEEP * 32 + lane; c < size; c += 32) dst[c] *= mul;
+    }
 }
 
 // A sequence's record becomes its last taps - 1 projections (after a step of several rows).  A step of fewer rows than
@@ -261,7 +312,7 @@ static int launch_delta_step(SbDelta p, SbBatch batch, void* y, cudaStream_t str
 
 extern "C" {
 
-// p [rows, 2 G D + H V], rows ld apart; w [channels, taps]; state [slots][taps - 1][channels] floats; out [rows, channels]
+// p [rows, 2 G D + H V], rows ld apart; w [taps, channels]; state [slots][taps - 1][channels] floats; out [rows, channels]
 // floats.  one_row: every sequence of the step brings one row (the record is moved on in the same kernel).
 int sb_conv_unit_heads(int dtype, const void* p, long long ld, const float* w, int taps, float* state, long long state_slot, SbBatch batch,
                        int G, int D, int H, int V, float q_scale, float* out, const float* inner, long long inner_ld, int n_inner,
@@ -269,20 +320,27 @@ int sb_conv_unit_heads(int dtype, const void* p, long long ld, const float* w, i
     if (batch.n_rows <= 0) return 0;
     if (taps < 1 || (taps > 1 && state == nullptr) || D < 1 || V < 1 || n_inner > low_ld) return (int)cudaErrorInvalidValue;
     typedef __nv_bfloat16 bf;
-    const bool advance = one_row && taps > 1;
-    const long long warps = (long long)batch.n_rows * (2 * G + H + 1);
+    const bool advance = one_row && taps > 1 && batch.n_rows < 512;
+    const int R = batch.n_rows >= 512 ? 4 : 1;   // few rows: a warp each, so that they spread over the SMs
+    const long long warps = (long long)((batch.n_rows + R - 1) / R) * (2 * G + H + 1);
+    if (warps > 0x7fffffffll) return (int)cudaErrorInvalidValue;
     const int per_block = batch.n_rows < 64 ? 2 : 8;
     const unsigned int blocks = (unsigned int)((warps + per_block - 1) / per_block);
-#define SB_CU(T, A)                                                                                                            \
-    sb_launch(conv_unit_heads_kernel<T, A>, blocks, per_block * 32, 0, stream, (const T*)p, ld, w, taps, state, state_slot, batch, G, D, H, \
-              V, q_scale, out, inner, inner_ld, n_inner, (T*)low, low_ld)
-    if (dtype == SB_F32) {
-        if (advance) SB_CU(float, true);
-        else SB_CU(float, false);
-    } else {
-        if (advance) SB_CU(bf, true);
-        else SB_CU(bf, false);
-    }
+#define SB_CU(T, R, A, N)                                                                                                      \
+    sb_launch(conv_unit_heads_kernel<T, R, A, N>, blocks, per_block * 32, 0, stream, (const T*)p, ld, w, taps, state, state_slot, batch, G, D, \
+              H, V, q_scale, out, inner, inner_ld, n_inner, (T*)low, low_ld)
+#define SB_CUT(T)                                      \
+    do {                                               \
+        if (advance && R == 1) SB_CU(T, 1, true, 0);   \
+        else if (R == 1) SB_CU(T, 1, false, 0);        \
+        else if (taps == 4) SB_CU(T, 4, false, 4);     \
+        else if (taps == 3) SB_CU(T, 4, false, 3);     \
+        else if (taps == 2) SB_CU(T, 4, false, 2);     \
+        else SB_CU(T, 4, false, 0);                    \
+    } while (0)
+    if (dtype == SB_F32) SB_CUT(float);
+    else SB_CUT(bf);
+#undef SB_CUT
 #undef SB_CU
     if (taps > 1 && !advance) {
         const int C = 2 * G * D + H * V;

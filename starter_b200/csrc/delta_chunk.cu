@@ -20,25 +20,45 @@
 
 #define DC 16             // tokens of a chunk
 #define DC_THREADS 128
+#define DC_STAGES 4       // chunks whose operands are in shared memory or on their way
 
 // One (chunk, head) of the workspace, in floats: [DP][2 DC] columns W | q c, then [DC][DP] keys carried to the end, then
-// [DP] c_16, [DC][DC] P, [DC][VP] M V.  DP, VP: the head sizes rounded up to multiples of 4.
-__host__ __device__ __forceinline__ int dc_pad(int n) { return (n + 3) & ~3; }
-__host__ __device__ __forceinline__ long long dc_shared_part(int DP) { return (long long)(3 * DC + 1) * DP + DC * DC; }
+// [DP] c_16, [DC][DC] P, [DC][VP] M V.  DP: the key channels rounded up to 32, 64 or 128; VP: the value columns rounded up
+// to a multiple of 4.
+__host__ __device__ __forceinline__ int dc_key_pad(int n) { return n <= 32 ? 32 : (n <= 64 ? 64 : 128); }
+__host__ __device__ __forceinline__ int dc_value_pad(int n) { return (n + 3) & ~3; }
+__host__ __device__ constexpr int dc_shared_part(int DP) { return (3 * DC + 1) * DP + DC * DC; }
 __host__ __device__ __forceinline__ long long dc_cell(int DP, int VP) { return dc_shared_part(DP) + (long long)DC * VP; }
 // First chunk of sequence s in the workspace; rows / DC + n_seqs places hold every step's chunks.
 __device__ __forceinline__ int dc_base(const SbBatch& b, int s) { return b.cu_q[s] / DC + s; }
 
-__global__ void __launch_bounds__(DC_THREADS)
-delta_chunk_prepare_kernel(SbDelta p, SbBatch batch, float* __restrict__ ws, int DP, int VP) {
-    extern __shared__ float sm[];
-    const int D = p.D, V = p.V, G = p.G, H = p.H, LD = DP + 4;
+// row i of M times the sixteen values x (M is lower triangular)
+__device__ __forceinline__ float dc_row_times(const float* m, int i, const float (&x)[DC]) {
+    float sum = 0.f;
+#pragma unroll
+    for (int j = 0; j < DC; j += 4)
+        if (j <= i) {
+            const float4 r = *reinterpret_cast<const float4*>(m + i * DC + j);
+            sum = fmaf(r.x, x[j], sum);
+            sum = fmaf(r.y, x[j + 1], sum);
+            sum = fmaf(r.z, x[j + 2], sum);
+            sum = fmaf(r.w, x[j + 3], sum);
+        }
+    return sum;
+}
+
+template <int DP>
+__global__ void __launch_bounds__(DC_THREADS, DP == 128 ? 4 : 6)
+delta_chunk_prepare_kernel(SbDelta p, SbBatch batch, float* __restrict__ ws, int VP) {
+    constexpr int LD = DP + 4, E = DP / 16;
+    extern __shared__ __align__(16) float sm[];
     float* qs = sm;               // [DC][LD]
     float* ks = qs + DC * LD;
     float* gs = ks + DC * LD;
-    __shared__ float As[DC][DC + 1], Ms[DC][DC + 1], bs[DC];
-    __shared__ __align__(16) float Ps[DC * DC];
+    __shared__ float As[DC][DC + 1], bs[DC];
+    __shared__ __align__(16) float Ms[DC * DC], Ps[DC * DC];
     __shared__ int s_seq;
+    const int D = p.D, V = p.V, G = p.G, H = p.H;
     const int head = blockIdx.y, tid = threadIdx.x;
     const float neg_rate = -expf(p.a_log[head]);
     pdl_wait();
@@ -57,7 +77,7 @@ delta_chunk_prepare_kernel(SbDelta p, SbBatch batch, float* __restrict__ ws, int
     if (nt <= 0) return;
     const int kvh = head / (H / G), C = 2 * G * D + H * V;
     for (int e = tid; e < DC * DP; e += DC_THREADS) {
-        const int t = e / DP, d = e - t * DP;
+        const int t = e / DP, d = e % DP;
         float q = 0.f, k = 0.f, g = 1.f;
         if (t < nt && d < D) {
             const float* in = p.qkv + (long long)(row0 + t) * C;
@@ -74,25 +94,23 @@ delta_chunk_prepare_kernel(SbDelta p, SbBatch batch, float* __restrict__ ws, int
     __syncthreads();
     {   // A and P: sixteen lanes per key j (and 15 - j after it), each with every 16th channel
         const int group = tid >> 4, l = tid & 15;
+        const unsigned int half_mask = 0xffffu << (tid & 16);   // the two groups of a warp have loops of different lengths
 #pragma unroll 1
         for (int half = 0; half < 2; ++half) {
             const int j = half == 0 ? group : DC - 1 - group;
-            float kd[8];   // k_j times the decays since token j
+            float kd[E];   // k_j times the decays since token j
 #pragma unroll
-            for (int e = 0; e < 8; ++e) kd[e] = l + 16 * e < DP ? ks[j * LD + l + 16 * e] : 0.f;
+            for (int e = 0; e < E; ++e) kd[e] = ks[j * LD + l + 16 * e];
+#pragma unroll 1
             for (int i = j; i < DC; ++i) {
                 float a = 0.f, o = 0.f;
 #pragma unroll
-                for (int e = 0; e < 8; ++e) {
-                    const int d = l + 16 * e;
-                    if (d < DP) {
-                        if (i > j) kd[e] *= gs[i * LD + d];
-                        a = fmaf(ks[i * LD + d], kd[e], a);
-                        o = fmaf(qs[i * LD + d], kd[e], o);
-                    }
+                for (int e = 0; e < E; ++e) {
+                    const int at = i * LD + l + 16 * e;
+                    if (i > j) kd[e] *= gs[at];
+                    a = fmaf(ks[at], kd[e], a);
+                    o = fmaf(qs[at], kd[e], o);
                 }
-                // the two groups of a warp have loops of different lengths: shuffles name their own half
-                const unsigned int half_mask = 0xffffu << (tid & 16);
 #pragma unroll
                 for (int off = 8; off > 0; off >>= 1) {
                     a += __shfl_xor_sync(half_mask, a, off);
@@ -114,75 +132,95 @@ delta_chunk_prepare_kernel(SbDelta p, SbBatch batch, float* __restrict__ ws, int
 #pragma unroll
             for (int j = 0; j < i; ++j) sum = fmaf(As[i][j], t[j], sum);
             t[i] = (i == tid ? 1.0f : 0.f) - bs[i] * sum;
-            if (i < tid) t[i] = 0.f;
-            Ms[i][tid] = t[i] * bs[tid];
+            Ms[i * DC + tid] = t[i] * bs[tid];
         }
     }
     __syncthreads();
     float* cell = ws + ((long long)blockIdx.x * H + head) * dc_cell(DP, VP);
     float* wq = cell;
-    float* kh = wq + (long long)2 * DC * DP;
-    float* cg = kh + (long long)DC * DP;
+    float* kh = wq + 2 * DC * DP;
+    float* cg = kh + DC * DP;
     float* pg = cg + DP;
     float* mv = pg + DC * DC;
-    for (int d = tid; d < DP; d += DC_THREADS) {
-        float kc[DC], row[DC];
-        float c = 1.0f;
-#pragma unroll
-        for (int i = 0; i < DC; ++i) {
-            c *= gs[i * LD + d];
-            kc[i] = ks[i * LD + d] * c;
-            row[i] = qs[i * LD + d] * c;
-        }
-        cg[d] = c;
-        float4* dst = reinterpret_cast<float4*>(wq + (long long)d * 2 * DC);
-#pragma unroll
-        for (int i = 0; i < DC; i += 4) dst[(DC + i) / 4] = make_float4(row[i], row[i + 1], row[i + 2], row[i + 3]);
-#pragma unroll
-        for (int i = 0; i < DC; ++i) {
-            float w = 0.f;
-#pragma unroll
-            for (int j = 0; j <= i; ++j) w = fmaf(Ms[i][j], kc[j], w);
-            row[i] = w;
-        }
-#pragma unroll
-        for (int i = 0; i < DC; i += 4) dst[i / 4] = make_float4(row[i], row[i + 1], row[i + 2], row[i + 3]);
-        c = 1.0f;
-#pragma unroll
-        for (int j = DC - 1; j >= 0; --j) {
-            kh[(long long)j * DP + d] = ks[j * LD + d] * c;
-            c *= gs[j * LD + d];
-        }
-    }
     for (int e = tid; e < DC * DC; e += DC_THREADS) pg[e] = Ps[e];
-    for (int col = tid; col < VP; col += DC_THREADS) {
-        float v[DC];
+#pragma unroll 1
+    for (int item = tid; item < DP + VP; item += DC_THREADS) {   // a key channel, or a value column
+        float x[DC];
+        if (item < DP) {
+            const int d = item;
+            float4* dst = reinterpret_cast<float4*>(wq + (long long)d * 2 * DC);
+            float c = 1.0f;
 #pragma unroll
-        for (int t = 0; t < DC; ++t)
-            v[t] = t < nt && col < V ? p.qkv[(long long)(row0 + t) * C + 2 * G * D + head * V + col] : 0.f;
+            for (int j = DC - 1; j >= 0; --j) {
+                kh[j * DP + d] = ks[j * LD + d] * c;
+                c *= gs[j * LD + d];
+            }
+            cg[d] = c;
+            c = 1.0f;
 #pragma unroll
-        for (int i = 0; i < DC; ++i) {
-            float u = 0.f;
+            for (int i = 0; i < DC; ++i) {
+                c *= gs[i * LD + d];
+                x[i] = qs[i * LD + d] * c;
+            }
 #pragma unroll
-            for (int j = 0; j <= i; ++j) u = fmaf(Ms[i][j], v[j], u);
-            mv[(long long)i * VP + col] = u;
+            for (int i = 0; i < DC; i += 4) dst[(DC + i) / 4] = make_float4(x[i], x[i + 1], x[i + 2], x[i + 3]);
+            c = 1.0f;
+#pragma unroll
+            for (int i = 0; i < DC; ++i) {
+                c *= gs[i * LD + d];
+                x[i] = ks[i * LD + d] * c;
+            }
+#pragma unroll
+            for (int i = 0; i < DC; i += 4)
+                dst[i / 4] = make_float4(dc_row_times(Ms, i, x), dc_row_times(Ms, i + 1, x), dc_row_times(Ms, i + 2, x), dc_row_times(Ms, i + 3, x));
+        } else {
+            const int col = item - DP;
+#pragma unroll
+            for (int t = 0; t < DC; ++t)
+                x[t] = t < nt && col < V ? p.qkv[(long long)(row0 + t) * C + 2 * G * D + head * V + col] : 0.f;
+#pragma unroll
+            for (int i = 0; i < DC; ++i) mv[(long long)i * VP + col] = dc_row_times(Ms, i, x);
         }
     }
 }
 
+// CT floats from or to 16- or 8-byte aligned shared memory.
+template <int CT> __device__ __forceinline__ void dc_load(const float* p, float (&v)[CT]) {
+#pragma unroll
+    for (int c = 0; c < CT; c += 2) {
+        const float2 f = *reinterpret_cast<const float2*>(p + c);
+        v[c] = f.x;
+        v[c + 1] = f.y;
+    }
+}
+template <> __device__ __forceinline__ void dc_load<4>(const float* p, float (&v)[4]) {
+    const float4 f = *reinterpret_cast<const float4*>(p);
+    v[0] = f.x;
+    v[1] = f.y;
+    v[2] = f.z;
+    v[3] = f.w;
+}
+template <int CT> __device__ __forceinline__ void dc_store(float* p, const float (&v)[CT]) {
+#pragma unroll
+    for (int c = 0; c < CT; c += 2) *reinterpret_cast<float2*>(p + c) = make_float2(v[c], v[c + 1]);
+}
+template <> __device__ __forceinline__ void dc_store<4>(float* p, const float (&v)[4]) {
+    *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+}
+
 // A block of four warps per (sequence, head, 4 CT value columns); a warp owns CT columns of the state, of U and of O
-// throughout, so that inside a chunk only the shared operands (one cp.async stage ahead) need the block's barrier.
+// throughout, so that inside a chunk only the shared operands (DC_STAGES - 1 chunks ahead) need the block's barrier.
 // Product with the state: lane = (row tile of 4 among the 32 rows W | q c) + 8 * (share of the key channels); the four
-// shares meet by shuffles, each lane keeping one row.  NE: key channels per lane in the update (DP <= 32 NE).
-template <int CT, int NE>
+// shares meet by shuffles, each lane keeping one row.  What the chunk's later steps read of the operands is fetched into
+// registers first: the chain from one chunk's state to the next is what the time here consists of.
+template <int CT, int DP>
 __global__ void __launch_bounds__(DC_THREADS)
-delta_chunk_scan_kernel(SbDelta p, SbBatch batch, const float* __restrict__ ws, float* __restrict__ o_raw, int DP, int VP) {
+delta_chunk_scan_kernel(SbDelta p, SbBatch batch, const float* __restrict__ ws, float* __restrict__ o_raw, int VP) {
     extern __shared__ __align__(16) float smf[];
-    constexpr int VB = 4 * CT;
+    constexpr int VB = 4 * CT, NE = DP / 32, PART = dc_shared_part(DP), STAGE = PART + DC * VB;
     const int D = p.D, V = p.V, H = p.H;
-    const int part = (int)dc_shared_part(DP), stage = part + DC * VB;
-    float* buf = smf;                           // two stages: the cell's shared part, then [DC][VB] of M V
-    float* Ssm = buf + 2 * stage;               // [4 warps][DP][CT]
+    float* buf = smf;                           // the stages: a cell's shared part, then [DC][VB] of M V
+    float* Ssm = buf + DC_STAGES * STAGE;       // [4 warps][DP][CT]
     float* Usm = Ssm + 4 * DP * CT;             // [4 warps][DC][CT]
     const int s = blockIdx.x, head = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int j0 = blockIdx.z * VB, col0 = j0 + warp * CT;
@@ -197,47 +235,47 @@ delta_chunk_scan_kernel(SbDelta p, SbBatch batch, const float* __restrict__ ws, 
     for (int e = 0; e < NE; ++e) {
         const int d = e * 32 + lane;
 #pragma unroll
-        for (int c = 0; c < CT; ++c) {
-            S[e][c] = d < D && col0 + c < V ? Sg[(long long)d * V + col0 + c] : 0.f;
-            if (d < DP) Sw[d * CT + c] = S[e][c];
-        }
+        for (int c = 0; c < CT; ++c) S[e][c] = d < D && col0 + c < V ? Sg[(long long)d * V + col0 + c] : 0.f;
+        dc_store<CT>(Sw + d * CT, S[e]);
     }
     const long long cell = dc_cell(DP, VP), base = dc_base(batch, s);
-    auto fetch = [&](int chunk, int b) {
-        const float* src = ws + ((base + chunk) * H + head) * cell;
-        float* dst = buf + b * stage;
-        for (int e = tid; e < part / 4; e += DC_THREADS) cp_async_16(dst + e * 4, src + e * 4);
-        for (int e = tid; e < DC * VB / 4; e += DC_THREADS) {
-            const int t = e / (VB / 4), c = (e % (VB / 4)) * 4;
-            if (j0 + c < VP) cp_async_16(dst + part + t * VB + c, src + part + (long long)t * VP + j0 + c);
-            else *reinterpret_cast<float4*>(dst + part + t * VB + c) = make_float4(0.f, 0.f, 0.f, 0.f);
+    auto fetch = [&](int chunk) {               // always one group of copies, so that the waits count the same
+        if (chunk < chunks) {
+            const float* src = ws + ((base + chunk) * H + head) * cell;
+            float* dst = buf + (chunk % DC_STAGES) * STAGE;
+            for (int e = tid; e < PART / 4; e += DC_THREADS) cp_async_16(dst + e * 4, src + e * 4);
+            for (int e = tid; e < DC * VB / 4; e += DC_THREADS) {
+                const int t = e / (VB / 4), c = (e % (VB / 4)) * 4;
+                if (j0 + c < VP) cp_async_16(dst + PART + t * VB + c, src + PART + (long long)t * VP + j0 + c);
+                else *reinterpret_cast<float4*>(dst + PART + t * VB + c) = make_float4(0.f, 0.f, 0.f, 0.f);
+            }
         }
         cp_async_commit();
     };
-    fetch(0, 0);
+#pragma unroll
+    for (int c = 0; c < DC_STAGES - 1; ++c) fetch(c);
     const int rt = lane & 7, share = lane >> 3;
-    const int my = rt * 4 + (share >> 1) * 2 + (share & 1);      // the row among W | q c that this lane keeps
+    const int my = rt * 4 + share;              // the row among W | q c that this lane keeps
+    const bool is_u = my < DC;
     for (int ch = 0; ch < chunks; ++ch) {
-        const int b = ch & 1;
-        cp_async_wait<0>();
-        __syncthreads();                        // the stage is there, and nobody reads the other one any more
-        if (ch + 1 < chunks) fetch(ch + 1, b ^ 1);
-        const float* wq = buf + b * stage;
+        cp_async_wait<DC_STAGES - 2>();
+        __syncthreads();                        // the stage is there, and nobody reads the one before it any more
+        fetch(ch + DC_STAGES - 1);
+        const float* wq = buf + (ch % DC_STAGES) * STAGE;
         const float* kh = wq + 2 * DC * DP;
         const float* cg = kh + DC * DP;
         const float* pg = cg + DP;
-        const float* mv = buf + b * stage + part + warp * CT;
         float acc[4][CT];
 #pragma unroll
         for (int r = 0; r < 4; ++r)
 #pragma unroll
             for (int c = 0; c < CT; ++c) acc[r][c] = 0.f;
-#pragma unroll 4
-        for (int d = share; d < DP; d += 4) {
+#pragma unroll
+        for (int i = 0; i < DP / 4; ++i) {
+            const int d = i * 4 + share;
             const float4 a = *reinterpret_cast<const float4*>(wq + d * 2 * DC + rt * 4);
             float x[CT];
-#pragma unroll
-            for (int c = 0; c < CT; ++c) x[c] = Sw[d * CT + c];
+            dc_load<CT>(Sw + d * CT, x);
 #pragma unroll
             for (int c = 0; c < CT; ++c) {
                 acc[0][c] = fmaf(a.x, x[c], acc[0][c]);
@@ -246,6 +284,24 @@ delta_chunk_scan_kernel(SbDelta p, SbBatch batch, const float* __restrict__ ws, 
                 acc[3][c] = fmaf(a.w, x[c], acc[3][c]);
             }
         }
+        float kr[NE][DC], pr[DC], first[CT];    // this lane's keys, its row of P, its row of M V
+#pragma unroll
+        for (int e = 0; e < NE; ++e) {
+            const float keep = cg[e * 32 + lane];
+#pragma unroll
+            for (int t = 0; t < DC; ++t) kr[e][t] = kh[t * DP + e * 32 + lane];
+#pragma unroll
+            for (int c = 0; c < CT; ++c) S[e][c] *= keep;
+        }
+#pragma unroll
+        for (int t = 0; t < DC; t += 4) {
+            const float4 r = *reinterpret_cast<const float4*>(pg + (my & (DC - 1)) * DC + t);
+            pr[t] = r.x;
+            pr[t + 1] = r.y;
+            pr[t + 2] = r.z;
+            pr[t + 3] = r.w;
+        }
+        dc_load<CT>(buf + (ch % DC_STAGES) * STAGE + PART + (my & (DC - 1)) * VB + warp * CT, first);
         float mine[CT];
         {
             const bool up = share & 2, odd = share & 1;
@@ -255,57 +311,30 @@ delta_chunk_scan_kernel(SbDelta p, SbBatch batch, const float* __restrict__ ws, 
                 const float keep0 = (up ? acc[2][c] : acc[0][c]) + __shfl_xor_sync(0xffffffffu, send0, 16);
                 const float keep1 = (up ? acc[3][c] : acc[1][c]) + __shfl_xor_sync(0xffffffffu, send1, 16);
                 mine[c] = (odd ? keep1 : keep0) + __shfl_xor_sync(0xffffffffu, odd ? keep0 : keep1, 8);
+                first[c] -= mine[c];
             }
         }
-        if (my < DC) {
-#pragma unroll
-            for (int c = 0; c < CT; ++c) Uw[my * CT + c] = mv[my * VB + c] - mine[c];
-        }
+        if (is_u) dc_store<CT>(Uw + my * CT, first);
         __syncwarp();
-        if (my >= DC) {                         // this lane's row of O
-            const int i = my - DC;
-            const float* pr = pg + i * DC;
-#pragma unroll
-            for (int t = 0; t < DC; ++t) {
-                const float w = pr[t];          // zero for t > i
-#pragma unroll
-                for (int c = 0; c < CT; ++c) mine[c] = fmaf(w, Uw[t * CT + c], mine[c]);
-            }
-            const int row = ch * DC + i;
-            if (row < n) {
-                float* o = o_raw + ((long long)(row0 + row) * H + head) * V + col0;
-#pragma unroll
-                for (int c = 0; c < CT; ++c)
-                    if (col0 + c < V) o[c] = mine[c];
-            }
-        }
-#pragma unroll
-        for (int e = 0; e < NE; ++e) {
-            const int d = e * 32 + lane;
-            const float keep = d < DP ? cg[d] : 0.f;
-#pragma unroll
-            for (int c = 0; c < CT; ++c) S[e][c] *= keep;
-        }
 #pragma unroll
         for (int t = 0; t < DC; ++t) {
             float u[CT];
+            dc_load<CT>(Uw + t * CT, u);
 #pragma unroll
-            for (int c = 0; c < CT; ++c) u[c] = Uw[t * CT + c];
+            for (int c = 0; c < CT; ++c) {
 #pragma unroll
-            for (int e = 0; e < NE; ++e) {
-                const int d = e * 32 + lane;
-                const float k = d < DP ? kh[t * DP + d] : 0.f;
-#pragma unroll
-                for (int c = 0; c < CT; ++c) S[e][c] = fmaf(k, u[c], S[e][c]);
+                for (int e = 0; e < NE; ++e) S[e][c] = fmaf(kr[e][t], u[c], S[e][c]);
+                mine[c] = fmaf(pr[t], u[c], mine[c]);     // P is zero above its diagonal
             }
         }
 #pragma unroll
-        for (int e = 0; e < NE; ++e) {
-            const int d = e * 32 + lane;
-            if (d < DP) {
+        for (int e = 0; e < NE; ++e) dc_store<CT>(Sw + (e * 32 + lane) * CT, S[e]);
+        const int row = ch * DC + my - DC;
+        if (!is_u && row < n) {
+            float* o = o_raw + ((long long)(row0 + row) * H + head) * V + col0;
 #pragma unroll
-                for (int c = 0; c < CT; ++c) Sw[d * CT + c] = S[e][c];
-            }
+            for (int c = 0; c < CT; ++c)
+                if (col0 + c < V) o[c] = mine[c];
         }
         __syncwarp();                           // the next chunk reads the columns that the other lanes wrote
     }
@@ -335,17 +364,24 @@ __global__ void delta_chunk_finish_kernel(const float* __restrict__ o_raw, SbDel
     for (int c = lane; c < V; c += 32) y[wid * V + c] = from_f<T>(o[c] * rstd * p.norm[c] * (1.0f / (1.0f + expf(-gate[c]))));
 }
 
-template <int CT, int NE>
-static int launch_chunk_scan(SbDelta p, SbBatch batch, const float* ws, float* o_raw, int DP, int VP, cudaStream_t stream) {
-    const size_t smem = (size_t)(2 * (dc_shared_part(DP) + DC * 4 * CT) + 4 * DP * CT + 4 * DC * CT) * sizeof(float);
-    if (smem > 48 * 1024) {
-        const cudaError_t err = cudaFuncSetAttribute(delta_chunk_scan_kernel<CT, NE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        if (err != cudaSuccess) return (int)err;
-    }
+template <int CT, int DP>
+static int launch_chunk_scan(SbDelta p, SbBatch batch, const float* ws, float* o_raw, int VP, cudaStream_t stream) {
+    const size_t smem = (size_t)(DC_STAGES * (dc_shared_part(DP) + DC * 4 * CT) + 4 * DP * CT + 4 * DC * CT) * sizeof(float);
+    const cudaError_t err = cudaFuncSetAttribute(delta_chunk_scan_kernel<CT, DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (err != cudaSuccess) return (int)err;
     const dim3 grid(batch.n_seqs, p.H, (p.V + 4 * CT - 1) / (4 * CT));
     if (grid.z > 65535) return (int)cudaErrorInvalidValue;
-    sb_launch(delta_chunk_scan_kernel<CT, NE>, grid, DC_THREADS, smem, stream, p, batch, ws, o_raw, DP, VP);
+    sb_launch(delta_chunk_scan_kernel<CT, DP>, grid, DC_THREADS, smem, stream, p, batch, ws, o_raw, VP);
     SB_LAUNCH_CHECK();
+}
+
+template <int DP>
+static int launch_chunks(SbDelta p, SbBatch batch, float* ws, float* o_raw, int columns, cudaStream_t stream) {
+    const int VP = dc_value_pad(p.V);
+    const size_t smem = (size_t)(3 * DC * (DP + 4)) * sizeof(float);
+    sb_launch(delta_chunk_prepare_kernel<DP>, dim3(batch.n_rows / DC + batch.n_seqs, p.H), DC_THREADS, smem, stream, p, batch, ws, VP);
+    if (columns == 8) return launch_chunk_scan<2, DP>(p, batch, ws, o_raw, VP, stream);
+    return launch_chunk_scan<4, DP>(p, batch, ws, o_raw, VP, stream);
 }
 
 extern "C" {
@@ -353,7 +389,7 @@ extern "C" {
 // Floats of workspace for a step of this shape, or -1 for heads the kernels do not take (more than 128 key channels).
 long long sb_delta_chunk_floats(int rows, int n_seqs, int H, int D, int V) {
     if (D < 1 || D > 128 || V < 1 || V > 4096) return -1;
-    return (long long)(rows / DC + n_seqs) * H * dc_cell(dc_pad(D), dc_pad(V));
+    return (long long)(rows / DC + n_seqs) * H * dc_cell(dc_key_pad(D), dc_value_pad(V));
 }
 
 // ws: sb_delta_chunk_floats(...) floats; o_raw [rows, H V] floats; columns: value columns per block, 8 or 16.
@@ -361,19 +397,10 @@ int sb_delta_chunk(int dtype, SbDelta p, SbBatch batch, float* ws, float* o_raw,
     if (batch.n_seqs <= 0 || batch.n_rows <= 0) return 0;
     if (p.D < 1 || p.D > 128 || p.V < 1 || p.V > 4096 || p.G < 1 || p.H % p.G || p.H > 65535 || (columns != 8 && columns != 16))
         return (int)cudaErrorInvalidValue;
-    const int DP = dc_pad(p.D), VP = dc_pad(p.V);
-    const size_t smem = (size_t)(3 * DC * (DP + 4)) * sizeof(float);
-    sb_launch(delta_chunk_prepare_kernel, dim3(batch.n_rows / DC + batch.n_seqs, p.H), DC_THREADS, smem, stream, p, batch, ws, DP, VP);
-    int err;
-    if (columns == 8) {
-        if (DP <= 32) err = launch_chunk_scan<2, 1>(p, batch, ws, o_raw, DP, VP, stream);
-        else if (DP <= 64) err = launch_chunk_scan<2, 2>(p, batch, ws, o_raw, DP, VP, stream);
-        else err = launch_chunk_scan<2, 4>(p, batch, ws, o_raw, DP, VP, stream);
-    } else {
-        if (DP <= 32) err = launch_chunk_scan<4, 1>(p, batch, ws, o_raw, DP, VP, stream);
-        else if (DP <= 64) err = launch_chunk_scan<4, 2>(p, batch, ws, o_raw, DP, VP, stream);
-        else err = launch_chunk_scan<4, 4>(p, batch, ws, o_raw, DP, VP, stream);
-    }
+    const int DP = dc_key_pad(p.D);
+    const int err = DP == 32 ? launch_chunks<32>(p, batch, ws, o_raw, columns, stream)
+                  : DP == 64 ? launch_chunks<64>(p, batch, ws, o_raw, columns, stream)
+                             : launch_chunks<128>(p, batch, ws, o_raw, columns, stream);
     if (err) return err;
     const long long warps = (long long)batch.n_rows * p.H;
     const unsigned int blocks = (unsigned int)((warps * 32 + 255) / 256);

@@ -1318,22 +1318,22 @@ class Ops:
 
     def conv_unit_heads(self, ctx, p, weight, state, kv_heads, dim, q_scale, inner, n_inner, inner_width):
         """p [rows, channels] = [q heads | k heads | v], ``kv_heads`` heads of ``dim`` for q and k: a short causal convolution
-        per channel (``weight`` [channels, taps], 32-bit; ``state`` [slots, taps - 1, channels] holds each sequence's last
+        per channel (``weight`` [taps, channels], 32-bit; ``state`` [slots, taps - 1, channels] holds each sequence's last
         inputs and is brought up to date), silu, and for q and k the unit length per head (q times ``q_scale``); 32-bit
         rows.  Beside them [rows, inner_width] in p's type: the first ``n_inner`` columns of ``inner`` (32-bit), then zeros.
         The value heads' number does not matter here: their channels are dealt out 128 at a time."""
         rows, C = p.shape
-        taps = weight.shape[1]
+        taps = weight.shape[0]
         V = C - 2 * kv_heads * dim
-        if (p.stride(1) != 1 or tuple(weight.shape) != (C, taps) or weight.dtype != torch.float32 or not weight.is_contiguous() or V < 1
+        if (p.stride(1) != 1 or tuple(weight.shape) != (taps, C) or weight.dtype != torch.float32 or not weight.is_contiguous() or V < 1
                 or inner.dtype != torch.float32 or inner.shape[0] != rows or inner.stride(1) != 1 or inner.shape[1] < n_inner):
-            raise KernelError("conv_unit_heads: rows of queries, keys and values, 32-bit [channels, taps] weights and inner vectors")
+            raise KernelError("conv_unit_heads: rows of queries, keys and values, 32-bit [taps, channels] weights and inner vectors")
         if taps > 1 and (state is None or state.dtype != torch.float32 or tuple(state.shape[1:]) != (taps - 1, C) or not state.is_contiguous()):
             raise KernelError(f"conv_unit_heads: the state is [slots, {taps - 1}, {C}] 32-bit numbers")
         piece = next((n for n in (128, 96, 64, 32) if V % n == 0), V)
         out = torch.empty((rows, C), dtype=torch.float32, device=p.device)
         low = torch.empty((rows, inner_width), dtype=p.dtype, device=p.device)
-        one_row = ctx.max_q_len == 1
+        one_row = ctx.max_q_len == 1 and rows < 512     # the kernel then moves the records on itself
         self._check(self.lib.sb_conv_unit_heads(_code(p.dtype), _ptr(p), p.stride(0), _ptr(weight), taps,
                                                 _ptr(state) if taps > 1 else None, state.stride(0) if taps > 1 else 0, self._batch(ctx),
                                                 kv_heads, dim, V // piece, piece, float(q_scale), _ptr(out), _ptr(inner), inner.stride(0),
@@ -1374,8 +1374,10 @@ class Ops:
         return y
 
     def delta_columns(self, n_seqs: int, heads: int, vdim: int) -> int:
-        """Value columns per block of the walk over chunks: 16, or 8 while that leaves SMs without a block."""
-        return 16 if n_seqs * heads * -(-vdim // 16) >= self.sm_count() else 8
+        """Value columns per block of the walk over chunks: 16, or 8 while that would leave a third of the SMs without a
+        block.  Measured on the mixer's 2,048 tokens (us, 8 / 16 columns): 64 blocks of 16: 300 / 326 and 327 / 356; 128
+        blocks: 477 / 444."""
+        return 16 if 3 * n_seqs * heads * -(-vdim // 16) >= 2 * self.sm_count() else 8
 
     def moe_route(self, h, router, correction, top, scale, bias=None, over_chosen=False):
         """(chosen int32 [rows, top], weight 32-bit [rows, top]) of softmax(h router^T + bias) (32-bit): the ``top`` largest

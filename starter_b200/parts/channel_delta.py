@@ -57,13 +57,13 @@ class ChannelDelta:
         outer[H * D:, ra:ra + rg] = weights["g2"]
         self.w_outer = self.ops.prepare_matrix(outer)
         self.w_o = self.ops.prepare_matrix(weights["o"])
-        self.conv = torch.cat([f32("q_conv"), f32("k_conv"), f32("v_conv")], dim=0).contiguous()
+        self.conv = torch.cat([f32("q_conv"), f32("k_conv"), f32("v_conv")], dim=0).t().contiguous()     # [taps, channels]
         self.a_log, self.dt_bias, self.norm = f32("A_log"), f32("dt_bias"), f32("norm")
 
     def cache_request(self):
         s = self.spec
         state = StateRequest((s.num_heads * s.head_dim * s.v_dim,))
-        return (state, StateRequest((s.taps - 1, self.conv.shape[0]))) if s.taps > 1 else state
+        return (state, StateRequest((s.taps - 1, self.conv.shape[1]))) if s.taps > 1 else state
 
     def prepare(self, cache) -> None:
         pass

@@ -415,14 +415,14 @@ class EmulatedOps:
         return torch.tanh(logits / cap) * cap
 
     def conv_unit_heads(self, ctx, p, weight, state, kv_heads, dim, q_scale, inner, n_inner, inner_width):
-        rows, taps = p.shape[0], weight.shape[1]
+        rows, taps = p.shape[0], weight.shape[0]
         y = torch.zeros(p.shape, dtype=torch.float32, device=p.device)
         for b in range(ctx.n_seqs):
             slot, r0, r1 = int(ctx.seq_slot[b]), int(ctx.cu_q[b]), int(ctx.cu_q[b + 1])
             past = state[slot].float() if taps > 1 else y.new_zeros((0, p.shape[1]))
             hist = torch.cat([past, p[r0:r1].float()], dim=0)
             for j in range(taps):
-                y[r0:r1] += weight[:, j].float()[None, :] * hist[j:j + (r1 - r0)]
+                y[r0:r1] += weight[j].float()[None, :] * hist[j:j + (r1 - r0)]
             if taps > 1:
                 state[slot] = hist[hist.shape[0] - (taps - 1):]
         y = y * torch.sigmoid(y)

@@ -315,13 +315,14 @@ def test_long_delta_sequences_keep_their_state(mode):
 
 
 @pytest.mark.parametrize("mode", MODES)
-def test_unequal_sequences_in_one_step(mode):
-    """Sequences of lengths around sixteen and its multiples in one step, then one token each, then unequal pieces again."""
+@pytest.mark.parametrize("lengths", [[1, 5, 15, 16, 17, 33, 48, 100], [301, 2, 250, 1, 7, 3, 65, 18]])
+def test_unequal_sequences_in_one_step(mode, lengths):
+    """Sequences of lengths around sixteen and its multiples (and a step of many rows) in one step, then one token each, then
+    unequal pieces again."""
     rt = runtime(mode)
     spec = delta_spec(H=3, G=1, D=32, V=36, taps=4)
     w = delta_weights(spec, 90)
     part = part_of(rt, spec, w)
-    lengths = [1, 5, 15, 16, 17, 33, 48, 100]
     seqs = [rand((n + 1 + 19 - i, 80), 100 + i) for i, n in enumerate(lengths)]
     cache = Cache([part.cache_request()], n_slots=8, max_tokens=64 * 24, dtype=rt.dtype, device="cuda")
     slots = [cache.alloc() for _ in seqs]
