@@ -498,8 +498,8 @@ def _siparax_raw(width, latent, delta, ff, vocab=32000):
     gated one over the first one's latents."""
     def layer(kind, extra=()):
         mixer = dict(latent, scale=(latent["dim"] + latent["rot_dim"]) ** -0.5,
-                     rot={"base": 500000.0, "dims": latent["rot_dim"],
-                          "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}, **dict(extra))
+                     rot={"base": 1000000.0, "dims": latent["rot_dim"],
+                          "scaling": {"factor": 4.0, "original": 8192, "fast": 24.0, "slow": 2.0}}, **dict(extra))
         return {"type": kind, "mixer": mixer}
     recurrent = {"type": "channel_delta", "mixer": dict(delta, conv=4)}
     kinds = [recurrent, layer("latent_attention_2"), layer("latent_attention"),

@@ -68,7 +68,7 @@ CASES = {
     # sizes the tensor-core kernels take
     "B": _model(300, 128, 1e-6, 50.0, [
         _with(_delta(4, 4, 64, 64, 4, 32, 32), 256),
-        _with(_pairs(8, 64, 32, 64, 96, 128, 10000.0, (8.0, 128, 32.0, 1.0)), 192),
+        _with(_pairs(2, 80, 48, 64, 96, 128, 10000.0, (8.0, 128, 24.0, 1.0)), 192),
         _with(_halves(4, 32, 32, 128, 64, 64, 1000000.0, (16.0, 256, 16.0, 2.0)), 128),
         _with(_halves(16, 48, 32, 64, 64, 64, 1000000.0, (16.0, 256, 16.0, 2.0), kv_from=2), 64)]),
     # no feed-forward anywhere but once, no cap, no stretch, single heads, one tap, widths that are no multiples of 8

@@ -399,10 +399,10 @@ def plain_latent(h, w, s, rows=None):
 
 LATENT_SIZES = [
     dict(H=5, D=24, R=12, V=20, rq=28, rk=44),                                    # the general kernel
-    dict(H=8, D=64, R=32, V=64, rq=96, rk=128, base=10000.0),                     # sizes the tensor-core kernels take
+    dict(H=2, D=80, R=48, V=64, rq=96, rk=128, base=10000.0),                     # sizes the tensor-core kernels take
     dict(H=16, D=128, R=64, V=128, rq=64, rk=256, stretch=None),
     dict(H=1, D=10, R=2, V=6, rq=12, rk=14, base=100.0, stretch=None),
-    dict(H=4, D=32, R=16, V=48, rq=40, rk=64, base=500000.0, stretch=dict(factor=16.0, original=128.0, fast=32.0, slow=1.0), scale=0.3),
+    dict(H=6, D=40, R=8, V=56, rq=72, rk=64, base=300000.0, stretch=dict(factor=16.0, original=128.0, fast=24.0, slow=2.0), scale=0.3),
     dict(H=3, D=5, R=6, V=7, rq=11, rk=13),
 ]
 
