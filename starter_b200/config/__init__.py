@@ -6,7 +6,7 @@ from .specs import (ActMLPSpec, AttentionSpec, BiasedAttentionSpec, BlockSpec, B
                     SinusoidSpec, TalkingAttentionSpec, DiffAttentionSpec, GatedMLPSpec, GLASpec, GroupedNormSpec,
                     LatentAttentionSpec, ModelSpec, MoESpec, NormSpec, PairRopeSpec, ParallelBlockSpec, RopeSpec,
                     ScaledHalfRopeSpec, StreamBlockSpec, StreamNormSpec, WKVSpec, KeyValueAttentionSpec, MLSTMSpec, PairMixerSpec,
-                    SandwichBlockSpec, LoopSpec, LayerNormSpec, ChannelDeltaSpec)
+                    SandwichBlockSpec, LoopSpec, LayerNormSpec, ChannelDeltaSpec, LightningSpec, Mamba2Spec)
 
 __all__ = ["ConfigError", "ModelConfig", "TensorNames", "architecture_names", "config_from_dict", "load_config",
            "register_architecture", "save_config", "AttentionSpec", "BlockSpec", "GatedMLPSpec", "ModelSpec",
@@ -14,4 +14,4 @@ __all__ = ["ConfigError", "ModelConfig", "TensorNames", "architecture_names", "c
            "ParallelBlockSpec", "WKVSpec", "DiffAttentionSpec", "GLASpec", "MoESpec", "ScaledHalfRopeSpec", "StreamBlockSpec",
            "StreamNormSpec", "ActMLPSpec", "BranchNormSpec", "CausalConvSpec", "PostNormBlockSpec", "SinusoidSpec",
            "TalkingAttentionSpec", "KeyValueAttentionSpec", "MLSTMSpec", "PairMixerSpec", "SandwichBlockSpec", "LoopSpec",
-           "LayerNormSpec", "ChannelDeltaSpec"]
+           "LayerNormSpec", "ChannelDeltaSpec", "LightningSpec", "Mamba2Spec"]

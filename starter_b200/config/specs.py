@@ -58,7 +58,10 @@ class LayerNormSpec:
 class PairRopeSpec:
     """Rotary position encoding over neighbouring columns: (2j, 2j + 1) of the first ``rotary_dim`` columns turn
     by angle(p, j) = p * theta**(-2j / rotary_dim); angles, sines and the rotation itself are 32-bit.  With ``factor``
-    the frequencies are stretched by wavelength as ScaledHalfRopeSpec says."""
+    the frequencies are stretched by wavelength: with ``fast`` and ``slow`` as ScaledHalfRopeSpec says; with ``low`` and
+    ``high`` a pair whose wavelength l = 2 pi / f is longer than original / low turns ``factor`` times slower, one shorter
+    than original / high keeps f, and in between f becomes (1 - s) f / factor + s f with
+    s = (original / l - low) / (high - low); cosines and sines are not scaled then."""
 
     theta: float
     rotary_dim: int
@@ -66,6 +69,8 @@ class PairRopeSpec:
     original: Optional[float] = None
     fast: Optional[float] = None
     slow: Optional[float] = None
+    low: Optional[float] = None
+    high: Optional[float] = None
     kind: str = "rope_pairs"
 
 
@@ -75,7 +80,7 @@ class ScaledHalfRopeSpec:
     i + rotary_dim/2, with 32-bit angles taken in the kernels (no table) and, when ``factor`` is given, frequencies
     stretched by wavelength: with d(t) = rotary_dim ln(original / (2 pi t)) / (2 ln theta), pairs below d(fast) keep
     f_i = theta**(-2i / rotary_dim), pairs above d(slow) turn ``factor`` times slower, a linear ramp in between, and
-    cosines and sines grow by 0.1 ln(factor) + 1."""
+    cosines and sines grow by 0.1 ln(factor) + 1.  With ``low`` and ``high`` instead: as PairRopeSpec says."""
 
     theta: float
     rotary_dim: int
@@ -83,6 +88,8 @@ class ScaledHalfRopeSpec:
     original: Optional[float] = None
     fast: Optional[float] = None
     slow: Optional[float] = None
+    low: Optional[float] = None
+    high: Optional[float] = None
     kind: str = "rope_half_scaled"
 
 
@@ -188,7 +195,8 @@ class DiffAttentionSpec:
     queries and keys hold [map 1 | map 2] of ``head_dim`` columns each, every map is a softmax attention of its own, and
     a head's output is (a1 - lambda a2) divided by its root mean square over ``v_dim`` (eps ``norm_eps``) times
     (1 - ``diff``), with lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + ``diff`` from four learned vectors.  ``window``:
-    only the last ``window`` keys are visible (None: all); ``position``: a position part applied to every map;
+    only the last ``window`` keys are visible (None: all); ``chunk``: key j is visible to query i only if
+    i // chunk == j // chunk (counted from the sequence's start); ``position``: a position part applied to every map;
     ``gate``: the heads' outputs, side by side, are multiplied element by element with sigmoid(W_g h) before the
     output projection."""
 
@@ -203,6 +211,7 @@ class DiffAttentionSpec:
     window: Optional[int] = None
     position: Optional[Any] = None
     gate: bool = False
+    chunk: Optional[int] = None
     kind: str = "diff_attention"
 
 
@@ -308,6 +317,45 @@ class ChannelDeltaSpec:
 
 
 @dataclass(frozen=True)
+class LightningSpec:
+    """Lightning attention (kind "lightning"): per head a [head_dim, v_dim] state S <- decay_h S + k_t v_t^T read as
+    o_t = S^T q_t, with a constant ``decay`` per head and q, k, v = silu of their projections (nothing is scaled).  The
+    concatenated heads are RMS-normed together (``norm_eps``, a weight over all heads' columns), multiplied by
+    sigmoid(W_g h) and projected."""
+
+    hidden_size: int
+    num_heads: int
+    head_dim: int
+    v_dim: int
+    decay: Tuple[float, ...]
+    norm_eps: float
+    kind: str = "lightning"
+
+
+@dataclass(frozen=True)
+class Mamba2Spec:
+    """A Mamba-2 layer (kind "mamba2"; inner = num_heads * v_dim, N = ``state``, G = ``groups``): W_in h holds
+    [z: inner | x: inner | B: G N | C: G N | dt: heads].  x, B and C together pass a short causal convolution over time per
+    channel (``taps``, with a bias; not added to its input) and silu; dt = softplus(dt + dt_bias).  Per head, with the B
+    and C of group h // (heads / groups):
+
+        S <- exp(-exp(A_log_h) dt_h) S + dt_h B x_h^T;   y_h = S^T C + D_h x_h
+
+    y (heads side by side) times silu(z) is RMS-normed in ``norm_groups`` equal parts (``norm_eps``), times a weight over
+    all columns, and projected."""
+
+    hidden_size: int
+    num_heads: int
+    v_dim: int
+    state: int
+    groups: int
+    taps: int
+    norm_groups: int
+    norm_eps: float
+    kind: str = "mamba2"
+
+
+@dataclass(frozen=True)
 class LatentAttentionSpec:
     """Causal attention through low-rank latents (kind "latent_attention").
 
@@ -385,6 +433,11 @@ class MoESpec:
     weights are their s divided by the chosen ones' sum (+ 1e-20), times ``route_scale``.  ``shared``: a feed-forward
     that every token runs and that is added.
 
+    ``scores`` "sigmoid": s = sigmoid(router logits) in the softmax's place.  ``groups`` > 1: the outputs form this many
+    equal groups of neighbours, a group's score is the sum of its two largest s + correction, and only outputs of the
+    ``keep_groups`` best groups can be chosen.  ``shared_gate``: the shared feed-forward's output is multiplied by
+    sigmoid(W_sg h), one number per token.
+
     ``router_bias``: the router's logits take a learned bias.  ``correction`` False: the router has no correction
     vector.  ``over_chosen``: the ``top`` largest logits (+ correction) are chosen and the weights are the softmax over
     the chosen logits only (the same numbers as above, without the softmax over all outputs in between)."""
@@ -399,6 +452,10 @@ class MoESpec:
     router_bias: bool = False
     correction: bool = True
     over_chosen: bool = False
+    scores: str = "softmax"
+    groups: int = 1
+    keep_groups: int = 1
+    shared_gate: bool = False
     kind: str = "moe"
 
 

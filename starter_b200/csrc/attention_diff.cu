@@ -1,16 +1,22 @@
 // What the attention with two score maps per head needs beside the attention kernels themselves: the rotation of
 // queries and keys with the cache write, and the join of a head's two maps.
 //
-// Rotation ("rotate half"): of a head's first `rot` columns, column i turns with column i + rot / 2 by the angle
-// position * freqs[i]; angle, sine and cosine are 32-bit, and both are multiplied by `mag`.  Later columns pass.
+// Rotation: of a head's first `rot` columns, pair i turns by the angle position * freqs[i]: columns i and i + rot / 2
+// ("rotate half", `halves`), or the neighbours 2i and 2i + 1.  Angle, sine and cosine are 32-bit, and both are multiplied by
+// `mag`.  Later columns pass.
 //
 // Join: with a1, a2 the two maps' results of one head, o = a1 - lam * a2, then o / sqrt(mean(o^2) + eps) * post, and with
 // a gate (pre-activations [rows, H * V], a view of wider rows) times sigmoid(gate), element by element.
 #include "attention_flex.cuh"
 
 template <class T>
-__device__ __forceinline__ float turned(const T* src, int c, int rot, const float* cs, const float* sn) {
+__device__ __forceinline__ float turned(const T* src, int c, int rot, int halves, const float* cs, const float* sn) {
     const int half = rot >> 1;
+    if (!halves) {
+        if (c >= rot) return to_f<T>(src[c]);
+        const float own = to_f<T>(src[c]), other = to_f<T>(src[c ^ 1]);
+        return c & 1 ? own * cs[c >> 1] + other * sn[c >> 1] : own * cs[c >> 1] - other * sn[c >> 1];
+    }
     if (c < half) return to_f<T>(src[c]) * cs[c] - to_f<T>(src[c + half]) * sn[c];
     if (c < rot) return to_f<T>(src[c]) * cs[c - half] + to_f<T>(src[c - half]) * sn[c - half];
     return to_f<T>(src[c]);
@@ -20,9 +26,9 @@ __device__ __forceinline__ float turned(const T* src, int c, int rot, const floa
 // wider rows (row strides in elements, heads side by side); v [rows, v_heads * v_dim] likewise.  The turned queries go
 // to q_out (contiguous), the turned keys and the values to the row's place in the cache.
 template <class T>
-__global__ void rotate_half_store_kernel(const T* __restrict__ q, long long q_row, const T* __restrict__ k, long long k_row,
+__global__ void rotate_store_kernel(const T* __restrict__ q, long long q_row, const T* __restrict__ k, long long k_row,
                                          const T* __restrict__ v, long long v_row, T* __restrict__ q_out, SbBatch batch, SbFlex p,
-                                         const float* __restrict__ freqs, int rot, float mag, int nq, int* status) {
+                                         const float* __restrict__ freqs, int rot, float mag, int halves, int nq, int* status) {
     extern __shared__ float trig[];
     pdl_wait();
     const int row = blockIdx.x, D = p.k_dim, half = rot >> 1;
@@ -44,7 +50,7 @@ __global__ void rotate_half_store_kernel(const T* __restrict__ q, long long q_ro
         if (u < nq) {
             const T* src = q + row * q_row + (long long)u * D;
             T* dst = q_out + ((long long)row * nq + u) * D;
-            for (int c = threadIdx.x; c < D; c += blockDim.x) dst[c] = from_f<T>(turned<T>(src, c, rot, cs, sn));
+            for (int c = threadIdx.x; c < D; c += blockDim.x) dst[c] = from_f<T>(turned<T>(src, c, rot, halves, cs, sn));
         } else if (u < nq + p.n_kv_heads) {
             const int h = u - nq;
             const long long tok = flex_token(p, slot, pos, h);
@@ -54,7 +60,7 @@ __global__ void rotate_half_store_kernel(const T* __restrict__ q, long long q_ro
             }
             const T* src = k + row * k_row + (long long)h * D;
             T* dst = (T*)p.k + tok * D;
-            for (int c = threadIdx.x; c < D; c += blockDim.x) dst[c] = from_f<T>(turned<T>(src, c, rot, cs, sn));
+            for (int c = threadIdx.x; c < D; c += blockDim.x) dst[c] = from_f<T>(turned<T>(src, c, rot, halves, cs, sn));
         } else {
             const int h = u - nq - p.n_kv_heads;
             const long long tok = flex_value_token(p, flex_token(p, slot, pos, h * per), h * per);
@@ -97,9 +103,9 @@ __global__ void diff_combine_kernel(const T* __restrict__ a, T* __restrict__ out
 
 extern "C" {
 
-int sb_rotate_half_store(int dtype, const void* q, long long q_row, const void* k, long long k_row, const void* v, long long v_row,
-                         void* q_out, SbBatch batch, SbFlex p, const float* freqs, int rot, float mag, int nq, int* status,
-                         cudaStream_t stream) {
+int sb_rotate_store(int dtype, const void* q, long long q_row, const void* k, long long k_row, const void* v, long long v_row,
+                         void* q_out, SbBatch batch, SbFlex p, const float* freqs, int rot, float mag, int halves, int nq, int* status,
+                    cudaStream_t stream) {
     if (batch.n_rows <= 0) return 0;
     if (rot < 0 || rot % 2 || rot > p.k_dim || (rot > 0 && freqs == nullptr)) return (int)cudaErrorInvalidValue;
     const int threads = p.k_dim >= 128 || p.v_dim >= 128 ? 128 : 64;
@@ -109,11 +115,11 @@ int sb_rotate_half_store(int dtype, const void* q, long long q_row, const void* 
     dim3 grid(batch.n_rows, per_row);
     const size_t smem = (size_t)rot * sizeof(float);
     if (dtype == SB_F32)
-        sb_launch(rotate_half_store_kernel<float>, grid, threads, smem, stream, (const float*)q, q_row, (const float*)k, k_row,
-                  (const float*)v, v_row, (float*)q_out, batch, p, freqs, rot, mag, nq, status);
+        sb_launch(rotate_store_kernel<float>, grid, threads, smem, stream, (const float*)q, q_row, (const float*)k, k_row,
+                  (const float*)v, v_row, (float*)q_out, batch, p, freqs, rot, mag, halves, nq, status);
     else
-        sb_launch(rotate_half_store_kernel<__nv_bfloat16>, grid, threads, smem, stream, (const __nv_bfloat16*)q, q_row,
-                  (const __nv_bfloat16*)k, k_row, (const __nv_bfloat16*)v, v_row, (__nv_bfloat16*)q_out, batch, p, freqs, rot, mag, nq,
+        sb_launch(rotate_store_kernel<__nv_bfloat16>, grid, threads, smem, stream, (const __nv_bfloat16*)q, q_row,
+                  (const __nv_bfloat16*)k, k_row, (const __nv_bfloat16*)v, v_row, (__nv_bfloat16*)q_out, batch, p, freqs, rot, mag, halves, nq,
                   status);
     SB_LAUNCH_CHECK();
 }

@@ -10,6 +10,7 @@
 // The read-out needs no second pass over the new state: with S' = g * S, r = S'^T k and p = S'^T q,
 // o = p + (k . q) u, so one pass over S gives r and p, and one more writes the new state.
 // Convolution, silu, unit norms, decays, state, sums, the output's norm and gate are 32-bit in every run.
+#include "conv_record.cuh"
 #include "delta.cuh"
 
 // A warp per (R consecutive rows, head of q, k or v), so that the loads of R rows are in flight together.  p [rows, C] in the
@@ -123,20 +124,6 @@ __global__ void conv_unit_heads_kernel(const T* __restrict__ p, long long ld, co
         }
         for (int c = DS_KEEP * 32 + lane; c < size; c += 32) dst[c] *= mul;
     }
-}
-
-// A sequence's record becomes its last taps - 1 projections (after a step of several rows).  A step of fewer rows than
-// that keeps the later entries of the old record: a thread reads its channel's entries before it writes them.
-template <class T>
-__global__ void conv_unit_state_kernel(const T* __restrict__ p, long long ld, int taps, float* state, long long state_slot, SbBatch batch, int C) {
-    pdl_wait();
-    const int s = blockIdx.x, first = batch.cu_q[s], n = batch.cu_q[s + 1] - first, keep = taps - 1;
-    float* rec = state + (long long)batch.seq_slot[s] * state_slot;
-    for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < C; c += gridDim.y * blockDim.x)
-        for (int e = 0; e < keep; ++e) {
-            const int src = n - keep + e;
-            rec[(long long)e * C + c] = src >= 0 ? to_f<T>(p[(long long)(first + src) * ld + c]) : rec[(long long)(e + n) * C + c];
-        }
 }
 
 // One block of eight warps per (sequence, head): warp w takes the key channels w, w + 8, ...; a lane takes VEC
@@ -343,12 +330,7 @@ int sb_conv_unit_heads(int dtype, const void* p, long long ld, const float* w, i
 #undef SB_CUT
 #undef SB_CU
     if (taps > 1 && !advance) {
-        const int C = 2 * G * D + H * V;
-        const dim3 grid(batch.n_seqs, batch.n_seqs < 64 ? (C + 127) / 128 : 1);
-        if (dtype == SB_F32)
-            sb_launch(conv_unit_state_kernel<float>, grid, 128, 0, stream, (const float*)p, ld, taps, state, state_slot, batch, C);
-        else
-            sb_launch(conv_unit_state_kernel<bf>, grid, 128, 0, stream, (const bf*)p, ld, taps, state, state_slot, batch, C);
+        launch_conv_record(dtype, p, ld, taps, state, state_slot, batch, 2 * G * D + H * V, stream);
     }
     SB_LAUNCH_CHECK();
 }

@@ -5,6 +5,9 @@
 //   chosen = the `top` largest of s + correction;  weight = s / (sum of the chosen s + 1e-20) * scale
 //   y = base + sum over chosen e of weight_e * (e is an identity output ? h : down_e(act(gate_e h, up_e h)))
 //
+// Options: s = sigmoid(W_r h) in the softmax's place; the choice among the best groups of outputs only; rows of W_r behind
+// the outputs', whose products are handed on (a gate of the base: base * sigmoid(product)).
+//
 // A pair is (row, k): the k-th choice of a row.  Pairs of identity outputs read no matrix.  For many rows the pairs are
 // put in the order of their experts (a slot per pair), so that one grouped product per matrix serves the step; for a
 // few pairs each pair streams its expert's matrices through the kernels below (a warp per output column).
@@ -87,27 +90,53 @@ moe_logits_kernel(const T* __restrict__ h, const float* __restrict__ router, flo
     }
 }
 
+// Where the largest of n values in shared memory stands (of equals the lowest index; 0 when none is above -inf);
+// `skip_inf`: entries of +inf are out already.
+__device__ __forceinline__ int warp_best(const float* v, int n, int lane, bool skip_inf) {
+    float best = -INFINITY;
+    int at = 0x7fffffff;
+    for (int e = lane; e < n; e += 32)
+        if (v[e] > best && !(skip_inf && v[e] == INFINITY)) {
+            best = v[e];
+            at = e;
+        }
+    for (int o = 16; o > 0; o >>= 1) {
+        const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+        const int oa = __shfl_xor_sync(0xffffffffu, at, o);
+        if (ob > best || (ob == best && oa < at)) {
+            best = ob;
+            at = oa;
+        }
+    }
+    return at == 0x7fffffff ? 0 : at;
+}
+
 // One warp per row: softmax over all outputs, the `top` largest of score + correction (of equals the lowest index), and
 // their weights.  bias (or null) is added to the logits first; correction may be null.  over_chosen: the `top` largest
-// LOGITS (+ correction) are chosen and weighted by the softmax over the chosen logits alone.
+// LOGITS (+ correction) are chosen and weighted by the softmax over the chosen logits alone.  sigmoid: the scores are
+// sigmoid(logit).  groups > 1: n_out / groups neighbours form a group, its score is the sum of its two largest choice scores,
+// and the outputs of all but the `keep` best groups (of equals the first) count as -inf.  Rows of logits are ld apart.
 __global__ void __launch_bounds__(256)
 moe_choose_kernel(const float* __restrict__ logits, const float* __restrict__ correction, const float* __restrict__ bias,
-                  int over_chosen, int* __restrict__ chosen, float* __restrict__ weight, int rows, int n_out, int top, float scale) {
+                  int over_chosen, int* __restrict__ chosen, float* __restrict__ weight, int rows, int n_out, int ld, int top, float scale,
+                  int sigmoid, int groups, int keep) {
     extern __shared__ __align__(16) float route_sm[];
     pdl_wait();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const long long row = (long long)blockIdx.x * 8 + warp;
     if (row >= rows) return;
-    float* s_s = route_sm + (size_t)warp * 2 * n_out;   // scores
+    float* s_s = route_sm + (size_t)warp * (2 * n_out + (groups > 1 ? groups : 0));   // scores
     float* c_s = s_s + n_out;                           // choice scores; -inf once taken
-    const float* lr = logits + row * n_out;
+    const float* lr = logits + row * ld;
     float mx = -INFINITY;
     for (int e = lane; e < n_out; e += 32) {
         s_s[e] = bias != nullptr ? lr[e] + bias[e] : lr[e];
         mx = fmaxf(mx, s_s[e]);
     }
     mx = warp_max(mx);
-    if (!over_chosen) {
+    if (sigmoid) {
+        for (int e = lane; e < n_out; e += 32) s_s[e] = 1.0f / (1.0f + expf(-s_s[e]));
+    } else if (!over_chosen) {
         float sum = 0.f;
         for (int e = lane; e < n_out; e += 32) {
             const float w = expf(s_s[e] - mx);
@@ -120,25 +149,33 @@ moe_choose_kernel(const float* __restrict__ logits, const float* __restrict__ co
     }
     for (int e = lane; e < n_out; e += 32) c_s[e] = correction != nullptr ? s_s[e] + correction[e] : s_s[e];
     __syncwarp();
+    if (groups > 1) {
+        float* g_s = c_s + n_out;   // the groups' scores; +inf once kept
+        const int each = n_out / groups;
+        for (int g = lane; g < groups; g += 32) {
+            float first = -INFINITY, second = -INFINITY;
+            for (int e = g * each; e < (g + 1) * each; ++e) {
+                const float c = c_s[e];
+                second = fmaxf(second, fminf(first, c));
+                first = fmaxf(first, c);
+            }
+            g_s[g] = each > 1 ? first + second : first;
+        }
+        __syncwarp();
+        for (int k = 0; k < keep; ++k) {
+            const int at = warp_best(g_s, groups, lane, true);
+            __syncwarp();
+            if (lane == 0) g_s[at] = INFINITY;
+            __syncwarp();
+        }
+        for (int e = lane; e < n_out; e += 32)
+            if (g_s[e / each] != INFINITY) c_s[e] = -INFINITY;
+        __syncwarp();
+    }
     float total = 0.f;
     int mine = 0;   // lane k keeps the k-th choice
     for (int k = 0; k < top; ++k) {
-        float best = -INFINITY;
-        int at = 0x7fffffff;
-        for (int e = lane; e < n_out; e += 32)
-            if (c_s[e] > best) {
-                best = c_s[e];
-                at = e;
-            }
-        for (int o = 16; o > 0; o >>= 1) {
-            const float ob = __shfl_xor_sync(0xffffffffu, best, o);
-            const int oa = __shfl_xor_sync(0xffffffffu, at, o);
-            if (ob > best || (ob == best && oa < at)) {
-                best = ob;
-                at = oa;
-            }
-        }
-        if (at == 0x7fffffff) at = 0;
+        const int at = warp_best(c_s, n_out, lane, false);
         if (lane == k) mine = at;
         total += s_s[at];
         __syncwarp();
@@ -321,12 +358,12 @@ moe_pair_down_kernel(const T* __restrict__ act, const int* __restrict__ chosen, 
 }
 
 // y[row] = base[row] + sum_k weight[row][k] * (identity ? h[row] : down[place of pair (row, k)]), summed in 32-bit in
-// the order of k.  slot_of_pair null: a pair's result lies at the pair's own index.  VEC (bfloat16 rows whose width is
+// the order of k.  base_gate (or null): the row's base is multiplied by sigmoid(base_gate[row * gate_ld]) first.  slot_of_pair null: a pair's result lies at the pair's own index.  VEC (bfloat16 rows whose width is
 // a multiple of 8): eight columns per thread, 16-byte accesses.
 template <class T, bool VEC>
 __global__ void moe_combine_kernel(const T* __restrict__ h, const T* __restrict__ down, const T* __restrict__ base,
                                    const int* __restrict__ chosen, const float* __restrict__ weight, const int* __restrict__ slot_of_pair,
-                                   T* __restrict__ y, int top, int n_experts, int width) {
+                                   T* __restrict__ y, int top, int n_experts, int width, const float* __restrict__ base_gate, int gate_ld) {
     __shared__ int place_s[MOE_MAX_TOP];
     __shared__ float w_s[MOE_MAX_TOP];
     pdl_wait();
@@ -338,6 +375,7 @@ __global__ void moe_combine_kernel(const T* __restrict__ h, const T* __restrict_
         place_s[threadIdx.x] = (e < 0 || e >= n_experts) ? -1 : (slot_of_pair != nullptr ? slot_of_pair[pair] : (int)pair);
     }
     __syncthreads();
+    const float share = base_gate != nullptr ? 1.0f / (1.0f + expf(-base_gate[row * gate_ld])) : 1.0f;
     if (VEC) {
         typedef __nv_bfloat16 bf;
         for (int c = threadIdx.x * 8; c < width; c += blockDim.x * 8) {
@@ -352,8 +390,8 @@ __global__ void moe_combine_kernel(const T* __restrict__ h, const T* __restrict_
                 const float2 f = __bfloat1622float2(hh[e]), b = __bfloat1622float2(bh[e]);
                 hv[2 * e] = f.x;
                 hv[2 * e + 1] = f.y;
-                acc[2 * e] = b.x;
-                acc[2 * e + 1] = b.y;
+                acc[2 * e] = b.x * share;
+                acc[2 * e + 1] = b.y * share;
             }
             for (int k = 0; k < top; ++k) {
                 const int at = place_s[k];
@@ -380,7 +418,7 @@ __global__ void moe_combine_kernel(const T* __restrict__ h, const T* __restrict_
         }
     } else {
         for (int c = threadIdx.x; c < width; c += blockDim.x) {
-            float acc = base != nullptr ? to_f<T>(base[row * width + c]) : 0.f;
+            float acc = base != nullptr ? to_f<T>(base[row * width + c]) * share : 0.f;
             const float hv = to_f<T>(h[row * width + c]);
             for (int k = 0; k < top; ++k) {
                 const int at = place_s[k];
@@ -394,9 +432,12 @@ __global__ void moe_combine_kernel(const T* __restrict__ h, const T* __restrict_
 extern "C" {
 
 int sb_moe_route(int dtype, const void* h, const float* router, const float* correction, const float* bias, int over_chosen,
-                 float* logits, int* chosen, float* weight, int rows, int width, int n_out, int top, float scale,
-                 cudaStream_t stream) {
+                 float* logits, int* chosen, float* weight, int rows, int width, int n_out, int top, float scale, int sigmoid,
+                 int groups, int keep, int extra, cudaStream_t stream) {
     if (rows <= 0) return 0;
+    const int n_rows_out = n_out + extra;   // rows of the router: the outputs' and those behind them
+    if (groups < 1 || n_out % groups || keep < 1 || keep > groups || keep * (n_out / groups) < top || extra < 0)
+        return (int)cudaErrorInvalidValue;
     if (n_out < 1 || n_out > MOE_MAX_OUTPUTS || top < 1 || top > MOE_MAX_TOP || top > n_out) return (int)cudaErrorInvalidValue;
     int R = rows >= 1024 ? 8 : (rows >= 256 ? 4 : (rows >= 64 ? 2 : 1));
     while (R > 1 && (size_t)R * width * sizeof(float) > 96 * 1024) R >>= 1;
@@ -404,20 +445,25 @@ int sb_moe_route(int dtype, const void* h, const float* router, const float* cor
     if (smem > 200 * 1024) return (int)cudaErrorInvalidValue;
     // one row per block: the router's rows are spread over blocks of eight; several rows: a block stages them once and
     // its warps walk all the router's rows
-    dim3 grid((unsigned int)((rows + R - 1) / R), R == 1 ? (unsigned int)((n_out + 7) / 8) : 1u);
+    dim3 grid((unsigned int)((rows + R - 1) / R), R == 1 ? (unsigned int)((n_rows_out + 7) / 8) : 1u);
 #define SB_ROUTE(T)                                                                                                              \
     do {                                                                                                                         \
         if (smem > 48 * 1024) {                                                                                                  \
             const cudaError_t err = cudaFuncSetAttribute(moe_logits_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
             if (err != cudaSuccess) return (int)err;                                                                             \
         }                                                                                                                        \
-        sb_launch(moe_logits_kernel<T>, grid, 256, smem, stream, (const T*)h, router, logits, rows, width, n_out, R);            \
+        sb_launch(moe_logits_kernel<T>, grid, 256, smem, stream, (const T*)h, router, logits, rows, width, n_rows_out, R);            \
     } while (0)
     if (dtype == SB_F32) SB_ROUTE(float);
     else SB_ROUTE(__nv_bfloat16);
 #undef SB_ROUTE
-    sb_launch(moe_choose_kernel, (unsigned int)((rows + 7) / 8), 256, (size_t)16 * n_out * sizeof(float), stream, (const float*)logits,
-              correction, bias, over_chosen, chosen, weight, rows, n_out, top, scale);
+    const size_t choose = (size_t)8 * (2 * n_out + (groups > 1 ? groups : 0)) * sizeof(float);
+    if (choose > 48 * 1024) {
+        const cudaError_t err = cudaFuncSetAttribute(moe_choose_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)choose);
+        if (err != cudaSuccess) return (int)err;
+    }
+    sb_launch(moe_choose_kernel, (unsigned int)((rows + 7) / 8), 256, choose, stream, (const float*)logits, correction, bias, over_chosen,
+              chosen, weight, rows, n_out, n_rows_out, top, scale, sigmoid, groups, keep);
     SB_LAUNCH_CHECK();
 }
 
@@ -469,19 +515,20 @@ int sb_moe_pairs(int dtype, const void* h, const int* chosen, const void* w_gate
 }
 
 int sb_moe_combine(int dtype, const void* h, const void* down, const void* base, const int* chosen, const float* weight,
-                   const int* slot_of_pair, void* y, int rows, int top, int n_experts, int width, cudaStream_t stream) {
+                   const int* slot_of_pair, void* y, int rows, int top, int n_experts, int width, const float* base_gate, int gate_ld,
+                   cudaStream_t stream) {
     if (rows <= 0) return 0;
     if (top < 1 || top > MOE_MAX_TOP) return (int)cudaErrorInvalidValue;
     typedef __nv_bfloat16 bf;
     if (dtype == SB_F32)
         sb_launch(moe_combine_kernel<float, false>, rows, width >= 1024 ? 256 : 128, 0, stream, (const float*)h, (const float*)down,
-                  (const float*)base, chosen, weight, slot_of_pair, (float*)y, top, n_experts, width);
+                  (const float*)base, chosen, weight, slot_of_pair, (float*)y, top, n_experts, width, base_gate, gate_ld);
     else if (width % 8 == 0)
         sb_launch(moe_combine_kernel<bf, true>, rows, width >= 2048 ? 256 : (width >= 1024 ? 128 : 64), 0, stream, (const bf*)h,
-                  (const bf*)down, (const bf*)base, chosen, weight, slot_of_pair, (bf*)y, top, n_experts, width);
+                  (const bf*)down, (const bf*)base, chosen, weight, slot_of_pair, (bf*)y, top, n_experts, width, base_gate, gate_ld);
     else
         sb_launch(moe_combine_kernel<bf, false>, rows, width >= 1024 ? 256 : 128, 0, stream, (const bf*)h, (const bf*)down,
-                  (const bf*)base, chosen, weight, slot_of_pair, (bf*)y, top, n_experts, width);
+                  (const bf*)base, chosen, weight, slot_of_pair, (bf*)y, top, n_experts, width, base_gate, gate_ld);
     SB_LAUNCH_CHECK();
 }
 

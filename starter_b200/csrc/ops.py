@@ -58,6 +58,13 @@ class SbDelta(Structure):
                 ("state", c_void_p), ("state_slot", c_longlong), ("H", c_int), ("G", c_int), ("D", c_int), ("V", c_int)]
 
 
+class SbDecay(Structure):
+    _fields_ = [("p", c_void_p), ("ld", c_longlong), ("q_col", c_int), ("k_col", c_int), ("v_col", c_int), ("act", c_int),
+                ("decay", c_void_p), ("log2_decay", c_void_p), ("dt", c_void_p), ("dt_ld", c_longlong), ("dt_bias", c_void_p),
+                ("rate", c_void_p), ("skip", c_void_p), ("state", c_void_p), ("state_slot", c_longlong), ("H", c_int), ("G", c_int),
+                ("D", c_int), ("V", c_int)]
+
+
 def _code(dtype: torch.dtype) -> int:
     if dtype == torch.float32:
         return F32
@@ -148,8 +155,8 @@ class Ops:
             "sb_embed_streams": [c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p],
             "sb_stream_norm": [c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
                                c_int, c_float, c_void_p],
-            "sb_rotate_half_store": [c_int, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, SbBatch,
-                                     SbFlex, c_void_p, c_int, c_float, c_int, c_void_p, c_void_p],
+            "sb_rotate_store": [c_int, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, SbBatch,
+                                SbFlex, c_void_p, c_int, c_float, c_int, c_int, c_void_p, c_void_p],
             "sb_diff_combine": [c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_void_p, c_longlong,
                                 c_void_p],
             "sb_mlstm_scan": [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_int, c_void_p,
@@ -168,13 +175,19 @@ class Ops:
             "sb_gla_scan": [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_float,
                             c_float, c_float, c_void_p, c_longlong, SbBatch, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p],
             "sb_moe_route": [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
-                             c_int, c_float, c_void_p],
+                             c_int, c_float, c_int, c_int, c_int, c_int, c_void_p],
             "sb_moe_sort": [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p],
             "sb_moe_gather": [c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
             "sb_moe_pairs": [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
                              c_float, c_float, c_int, c_void_p],
             "sb_moe_combine": [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
-                               c_int, c_void_p],
+                               c_int, c_void_p, c_int, c_void_p],
+            "sb_decay_step": [c_int, SbDecay, SbBatch, c_void_p, c_int, c_void_p],
+            "sb_decay_chunk": [SbDecay, SbBatch, c_void_p, c_void_p],
+            "sb_silu_columns": [c_int, c_void_p, c_longlong, c_int, c_int, c_void_p],
+            "sb_norm_gate": [c_int, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_int, c_void_p],
+            "sb_conv_silu": [c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_longlong, SbBatch, c_int, c_int, c_void_p,
+                             c_void_p],
             "sb_embed_sinusoid": [c_int, c_void_p, c_void_p, c_void_p, c_void_p, SbBatch, c_int, c_int, c_void_p, c_void_p],
             "sb_causal_conv": [c_int, c_void_p, c_void_p, c_void_p, c_longlong, SbBatch, c_int, c_int, c_void_p, c_void_p],
             "sb_branch_norm_add": [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p, c_float,
@@ -1118,26 +1131,26 @@ class Ops:
                                             float(eps), self._stream()), "stream_norm")
         return n
 
-    def rotate_half_store(self, ctx, q, k, v, layer_cache, freqs, rot, magnitude):
+    def rotate_store(self, ctx, q, k, v, layer_cache, freqs, rot, magnitude, halves):
         """q [rows, nq, D], k [rows, key heads, D] (views of wider rows, heads side by side) with the first ``rot`` columns
-        of every head turned (column i with column i + rot / 2) by position * ``freqs`` (32-bit, [rot / 2]), cosines and
-        sines times ``magnitude``; the turned keys and v [rows, value heads * value width] go to the layer's cache, the
+        of every head turned in pairs (``halves``: column i with column i + rot / 2; else columns 2i and 2i + 1) by
+        position * ``freqs`` (32-bit, [rot / 2]), cosines and sines times ``magnitude``; the turned keys and v [rows, value heads * value width] go to the layer's cache, the
         turned queries are returned [rows, nq, D]."""
         g = layer_cache.group
         rows, nq, D = q.shape
         if (D != g.request.head_dim or tuple(k.shape) != (rows, g.request.num_kv_heads, D) or v.shape[1] != g.v_heads * g.v_dim
                 or q.stride(2) != 1 or k.stride(2) != 1 or v.stride(1) != 1 or q.stride(1) != D or k.stride(1) != D
                 or not (q.dtype == k.dtype == v.dtype == layer_cache.k.dtype)):
-            raise KernelError("rotate_half_store: queries, keys or values do not fit the layer's cache")
+            raise KernelError("rotate_store: queries, keys or values do not fit the layer's cache")
         if freqs is None:
             rot = 0
         elif freqs.dtype != torch.float32 or freqs.numel() * 2 != rot or rot > D:
-            raise KernelError("rotate_half_store: one 32-bit frequency per pair of turned columns")
+            raise KernelError("rotate_store: one 32-bit frequency per pair of turned columns")
         p = self._flex(layer_cache)
         out = torch.empty((rows, nq, D), dtype=q.dtype, device=q.device)
-        self._check(self.lib.sb_rotate_half_store(_code(q.dtype), _ptr(q), q.stride(0), _ptr(k), k.stride(0), _ptr(v), v.stride(0),
-                                                  _ptr(out), self._batch(ctx), p, _ptr(freqs), int(rot), float(magnitude), nq,
-                                                  _ptr(ctx.status), self._stream()), "rotate_half_store")
+        self._check(self.lib.sb_rotate_store(_code(q.dtype), _ptr(q), q.stride(0), _ptr(k), k.stride(0), _ptr(v), v.stride(0),
+                                                  _ptr(out), self._batch(ctx), p, _ptr(freqs), int(rot), float(magnitude),
+                                             int(bool(halves)), nq, _ptr(ctx.status), self._stream()), "rotate_store")
         return out
 
     def diff_combine(self, a, heads, kv_heads, v_dim, lam, eps, post, gate=None):
@@ -1379,13 +1392,101 @@ class Ops:
         blocks: 477 / 444."""
         return 16 if 3 * n_seqs * heads * -(-vdim // 16) >= 2 * self.sm_count() else 8
 
-    def moe_route(self, h, router, correction, top, scale, bias=None, over_chosen=False):
+    # ---- a recurrence that decays by one number per head ------------------------------------
+
+    def conv_silu(self, ctx, u, weight, bias, state):
+        """silu(bias + sum_j weight[j] * u_(t - taps + 1 + j)) per sequence and channel, u [rows, channels] (a view of wider
+        rows will do), 32-bit sums, in u's type; ``weight`` [taps, channels] and ``bias`` are 32-bit, ``state`` [slots,
+        taps - 1, channels] holds each sequence's last inputs and is brought up to date."""
+        rows, C = u.shape
+        taps = weight.shape[0]
+        if (u.stride(1) != 1 or tuple(weight.shape) != (taps, C) or weight.dtype != torch.float32 or not weight.is_contiguous()
+                or bias.dtype != torch.float32 or bias.numel() != C or not bias.is_contiguous()):
+            raise KernelError("conv_silu: rows of channels, 32-bit [taps, channels] weights and a 32-bit bias")
+        if taps > 1 and (state is None or state.dtype != torch.float32 or tuple(state.shape[1:]) != (taps - 1, C) or not state.is_contiguous()):
+            raise KernelError(f"conv_silu: the state is [slots, {taps - 1}, {C}] 32-bit numbers")
+        out = torch.empty((rows, C), dtype=u.dtype, device=u.device)
+        one_row = ctx.max_q_len == 1     # the kernel then moves the records on itself
+        self._check(self.lib.sb_conv_silu(_code(u.dtype), _ptr(u), u.stride(0), _ptr(weight), _ptr(bias), taps,
+                                          _ptr(state) if taps > 1 else None, state.stride(0) if taps > 1 else 0, self._batch(ctx), C,
+                                          int(one_row), _ptr(out), self._stream()), "conv_silu")
+        if taps > 1 and not one_row:
+            self.launches += 1   # the record's kernel
+        return out
+
+    DECAY_CHUNK_MIN_ROWS = int(os.environ.get("STARTER_B200_DECAY_CHUNK_MIN", 16))   # a step whose longest sequence brings fewer rows walks them token by token
+
+    def decay_scan(self, ctx, p, q_col, k_col, v_col, state, heads, kv_heads, dim, vdim, decay=None, step=None, skip=None, silu=False):
+        """The recurrence S <- a S + w k v^T, o = S^T q + skip v per head over every sequence's rows, from and back into
+        ``state`` [slots, heads * dim * vdim]: p holds ``kv_heads`` queries of ``dim`` columns from q_col on, as many keys
+        from k_col on and ``heads`` values of ``vdim`` columns from v_col on; head h reads query and key
+        h // (heads / kv_heads).  ``decay`` [2, heads]: a constant a and its base-2 logarithm, w = 1; or ``step`` = (dt
+        [rows, heads], dt_bias, rate): w = softplus(dt + dt_bias), a = exp(-rate w); all 32-bit.  ``skip`` [heads] or None.
+        ``silu``: queries, keys and values pass silu first (in p itself, when the step is long).  Returns 32-bit
+        [rows, heads * vdim].  Steps of a few rows per sequence walk them token by token, longer ones in bfloat16 64 at a
+        time."""
+        rows = p.shape[0]
+        H, G, D, V = heads, kv_heads, dim, vdim
+        if (p.stride(1) != 1 or max(q_col + G * D, k_col + G * D, v_col + H * V) > p.shape[1] or H % G or (decay is None) == (step is None)
+                or state.dtype != torch.float32 or state.shape[1] != H * D * V or state.stride(1) != 1):
+            raise KernelError("decay_scan: queries, keys and values lie side by side in p; one kind of decay; a 32-bit state record")
+        dt, dt_bias, rate = step if step is not None else (None, None, None)
+        for t, n in ((decay, 2 * H), (dt_bias, H), (rate, H), (skip, H)):
+            if t is not None and (t.dtype != torch.float32 or t.numel() != n or not t.is_contiguous()):
+                raise KernelError("decay_scan: decays, step biases, rates and skips are 32-bit, one per head")
+        if dt is not None and (dt.dtype != torch.float32 or tuple(dt.shape) != (rows, H) or dt.stride(1) != 1):
+            raise KernelError("decay_scan: one 32-bit step size per row and head")
+        chunks = p.dtype == torch.bfloat16 and D <= 256 and ctx.max_q_len >= self.DECAY_CHUNK_MIN_ROWS
+        if silu and chunks:
+            if q_col != 0 or k_col != G * D or v_col != 2 * G * D:
+                raise KernelError("decay_scan: activated queries, keys and values are p's first columns")
+            self._check(self.lib.sb_silu_columns(_code(p.dtype), _ptr(p), p.stride(0), 2 * G * D + H * V, rows, self._stream()), "silu_columns")
+        out = torch.empty((rows, H * V), dtype=torch.float32, device=p.device)
+        a = SbDecay(_ptr(p), p.stride(0), int(q_col), int(k_col), int(v_col), int(bool(silu) and not chunks), _ptr(decay),
+                    _ptr(decay[1]) if decay is not None else None, _ptr(dt), dt.stride(0) if dt is not None else 0, _ptr(dt_bias), _ptr(rate),
+                    _ptr(skip), _ptr(state), state.stride(0), H, G, D, V)
+        if chunks:
+            self._check(self.lib.sb_decay_chunk(a, self._batch(ctx), _ptr(out), self._stream()), "decay_chunk")
+        else:
+            self._check(self.lib.sb_decay_step(_code(p.dtype), a, self._batch(ctx), _ptr(out), self.decay_columns(ctx.n_seqs, H, V),
+                                               self._stream()), "decay_step")
+        return out
+
+    def decay_columns(self, n_seqs: int, heads: int, vdim: int) -> int:
+        """Value columns per block of the token-by-token kernel: as many as leave two blocks per SM."""
+        for columns in (128, 64):
+            if vdim > columns // 2 and n_seqs * heads * -(-vdim // columns) >= 2 * self.sm_count():
+                return columns
+        return 32
+
+    def norm_gate(self, o, gate, weight, parts, eps, gate_first=False):
+        """32-bit rows o [rows, width] RMS-normed in ``parts`` equal consecutive parts, times ``weight`` (32-bit, per column)
+        and sigmoid(gate); ``gate_first``: o * silu(gate) is normed instead.  ``gate`` [rows, width] is a view of wider rows
+        in the type of the result."""
+        rows, width = o.shape
+        if (o.dtype != torch.float32 or not o.is_contiguous() or tuple(gate.shape) != (rows, width) or gate.stride(1) != 1
+                or weight.dtype != torch.float32 or weight.numel() != width or not weight.is_contiguous() or width % parts):
+            raise KernelError("norm_gate: contiguous 32-bit rows, a gate and a 32-bit weight per column")
+        y = torch.empty((rows, width), dtype=gate.dtype, device=o.device)
+        self._check(self.lib.sb_norm_gate(_code(gate.dtype), _ptr(o), _ptr(gate), gate.stride(0), _ptr(weight), _ptr(y), rows, width,
+                                          int(parts), float(eps), int(bool(gate_first)), self._stream()), "norm_gate")
+        return y
+
+    # ---- experts -----------------------------------------------------------------------------
+
+    def moe_route(self, h, router, correction, top, scale, bias=None, over_chosen=False, scores="softmax", groups=1, keep_groups=1,
+                  extra=0):
         """(chosen int32 [rows, top], weight 32-bit [rows, top]) of softmax(h router^T + bias) (32-bit): the ``top`` largest
         of score + correction, weighted by their scores over the chosen scores' sum, times ``scale``.  ``over_chosen``:
         the ``top`` largest logits (+ correction) instead, weighted by the softmax over the chosen logits alone.
-        ``correction`` and ``bias`` may be None."""
+        ``scores`` "sigmoid": sigmoid in the softmax's place.  ``groups``: the outputs form this many equal groups of
+        neighbours; only those of the ``keep_groups`` groups whose two largest score + correction sum highest can be
+        chosen.  ``extra``: the router's last rows are no outputs; their products are returned behind the weights, a view
+        [rows, extra].  ``correction`` and ``bias`` may be None."""
         rows, width = h.shape
-        n_out = router.shape[0]
+        n_out = router.shape[0] - extra
+        if scores not in ("softmax", "sigmoid") or (scores == "sigmoid" and over_chosen):
+            raise KernelError(f"moe_route: scores are 'softmax' or (not over the chosen logits alone) 'sigmoid', got {scores!r}")
         for extra in (correction, bias):
             if extra is not None and (extra.dtype != torch.float32 or extra.numel() != n_out or not extra.is_contiguous()):
                 raise KernelError(f"moe_route: correction and bias are {n_out} 32-bit numbers")
@@ -1394,17 +1495,17 @@ class Ops:
             raise KernelError("moe_route: a 32-bit router of up to 1024 outputs, up to 32 choices")
         chosen = torch.empty((rows, top), dtype=torch.int32, device=h.device)
         weight = torch.empty((rows, top), dtype=torch.float32, device=h.device)
-        logits = torch.empty((rows, n_out), dtype=torch.float32, device=h.device)
+        logits = torch.empty((rows, n_out + extra), dtype=torch.float32, device=h.device)
         self._check(self.lib.sb_moe_route(_code(h.dtype), _ptr(h), _ptr(router), _ptr(correction), _ptr(bias), int(bool(over_chosen)),
                                           _ptr(logits), _ptr(chosen), _ptr(weight), rows, width, n_out, int(top), float(scale),
-                                          self._stream()), "moe_route")
+                                          int(scores == "sigmoid"), int(groups), int(keep_groups), int(extra), self._stream()), "moe_route")
         self.launches += 1   # logits, then the choice
-        return chosen, weight
+        return (chosen, weight, logits[:, n_out:]) if extra else (chosen, weight)
 
     MOE_PAIRS_MAX = int(os.environ.get("STARTER_B200_MOE_PAIRS_MAX", 64))   # pairs up to which every pair streams its expert
 
-    def moe_experts(self, h, chosen, weight, w_gate_up, w_down, n_experts, alpha, limit, base):
-        """base + sum_k weight[:, k] * expert_chosen[:, k](h): experts are gated feed-forwards (the clamped activation with
+    def moe_experts(self, h, chosen, weight, w_gate_up, w_down, n_experts, alpha, limit, base, base_gate=None):
+        """base (times sigmoid(base_gate), 32-bit [rows, 1], when given) + sum_k weight[:, k] * expert_chosen[:, k](h): experts are gated feed-forwards (the clamped activation with
         its sigmoid factor ``alpha`` and ``limit``, or silu(gate) * up when ``alpha`` is None) with stacked
         matrices w_gate_up [experts, 2 ff, width] (gate over up) and w_down [experts, width, ff]; a choice >= n_experts
         is an identity output and adds weight * h.  A few pairs: each pair streams its expert's matrices (this library's
@@ -1441,9 +1542,12 @@ class Ops:
                                                   int(alpha is None), self._stream()),
                             "moe_pairs")
                 self.launches += 1
+        if base_gate is not None and (base is None or base_gate.dtype != torch.float32 or tuple(base_gate.shape) != (rows, 1)):
+            raise KernelError("moe_experts: one 32-bit gate per row of the base")
         y = torch.empty_like(h)
         self._check(self.lib.sb_moe_combine(dt, _ptr(h), _ptr(down), _ptr(base), _ptr(chosen), _ptr(weight), _ptr(slot_of_pair),
-                                            _ptr(y), rows, top, n_experts, width, self._stream()), "moe_combine")
+                                            _ptr(y), rows, top, n_experts, width, _ptr(base_gate),
+                                            base_gate.stride(0) if base_gate is not None else 0, self._stream()), "moe_combine")
         return y
 
     # ---- a layer whose branches read the 32-bit residual itself: position vector, short convolution, branch norm ----

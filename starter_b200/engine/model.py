@@ -138,11 +138,13 @@ class DecoderModel:
             x = self.embedding_norm.embed(ctx, tokens, self.embedding)   # normed 32-bit rows
         elif self.position is not None:
             x = self.position.embed(ctx, tokens, self.embedding)   # 32-bit rows with the positions' vectors added
+        elif self.spec.residual_float32 and self.spec.embedding_scale is not None:
+            x = ctx.ops.embed_streams(tokens, self.embedding, ctx.status, self.spec.embedding_scale, 1)   # 32-bit rows, scaled
         elif self.spec.residual_float32 and self.embedding.dtype != torch.float32:
             x = ctx.ops.embed(tokens, self.embedding, ctx.status, out_float32=True)   # the residual stays 32-bit
         else:
             x = ctx.ops.embed(tokens, self.embedding, ctx.status)
-        if self.spec.embedding_scale is not None:
+        if self.spec.embedding_scale is not None and not self.spec.residual_float32:
             x = (x.float() * self.spec.embedding_scale).to(x.dtype)
         if self.pass_starts:
             return self._hidden_in_passes(ctx, x)

@@ -1,7 +1,8 @@
 """Attention with two score maps per head over the same values (kind "diff_attention").
 
 Queries and keys hold two maps of ``head_dim`` columns per head, [map 1 | map 2]; every map is a causal softmax
-attention of its own (rotary positions, a sliding window), and a head's output is
+attention of its own (rotary positions in either layout of pairs, a sliding window or the query's own chunk), and a
+head's output is
 
     o = a1 - lambda * a2,   o / sqrt(mean(o^2) + eps) * (1 - diff),   lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff.
 
@@ -38,8 +39,10 @@ class DiffAttention:
         H, G, D = spec.num_heads, spec.num_kv_heads, spec.head_dim
         if H % G:
             raise ValueError(f"{H} query heads cannot share {G} key/value heads evenly")
-        if spec.window is not None and spec.window < 1:
-            raise ValueError(f"window must be a positive number of positions, got {spec.window}")
+        self.chunk = getattr(spec, "chunk", None)
+        for name, value in (("window", spec.window), ("chunk", self.chunk)):
+            if value is not None and value < 1:
+                raise ValueError(f"{name} must be a positive number of positions, got {value}")
         self.spec = spec
         self.ops = runtime.ops
         per = H // G
@@ -56,7 +59,8 @@ class DiffAttention:
 
     def cache_request(self):
         s = self.spec
-        return KVRequest(num_kv_heads=2 * s.num_kv_heads, head_dim=s.head_dim, window=s.window, v_dim=s.v_dim,
+        reach = [r for r in (s.window, self.chunk) if r is not None]     # how far back a query may look
+        return KVRequest(num_kv_heads=2 * s.num_kv_heads, head_dim=s.head_dim, window=min(reach) if reach else None, v_dim=s.v_dim,
                          v_heads=s.num_kv_heads)
 
     def prepare(self, cache) -> None:
@@ -70,9 +74,10 @@ class DiffAttention:
         nq, nk = 2 * H * D, 2 * G * D
         q = qkv[:, :nq].view(rows, 2 * H, D)
         k = qkv[:, nq:nq + nk].view(rows, 2 * G, D)
-        freqs, rot, mag = (None, 0, 1.0) if self.position is None else self.position.half_rotary()
-        q = ops.rotate_half_store(ctx, q, k, qkv[:, nq + nk:nq + nk + G * V], layer_cache, freqs, rot, mag)
-        a = ops.flex_attention(ctx, q, layer_cache, self.scale, v_dim=V, window=s.window)        # [rows, 2 H * V]
+        p = self.position
+        freqs, rot, mag, halves = (None, 0, 1.0, True) if p is None else (p.frequencies, p.rotary_dim, p.magnitude, p.halves)
+        q = ops.rotate_store(ctx, q, k, qkv[:, nq + nk:nq + nk + G * V], layer_cache, freqs, rot, mag, halves)
+        a = ops.flex_attention(ctx, q, layer_cache, self.scale, v_dim=V, chunk=self.chunk, window=s.window)        # [rows, 2 H * V]
         if self.gate:
             o = ops.diff_combine(a, H, G, V, self.lam, float(s.norm_eps), 1.0 - float(s.diff), gate=qkv[:, nq + nk + G * V:])
         else:

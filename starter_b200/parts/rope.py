@@ -48,12 +48,19 @@ class RotaryEmbedding:
 
 def stretched_frequencies(spec, device):
     """(32-bit frequencies [rotary_dim / 2] on the device, what multiplies cosines and sines) of a rotation over the first
-    ``rotary_dim`` columns; with ``factor`` the frequencies are stretched by wavelength (see ScaledHalfRopeSpec)."""
+    ``rotary_dim`` columns; with ``factor`` the frequencies are stretched by wavelength (see ScaledHalfRopeSpec, and
+    PairRopeSpec for ``low`` and ``high``)."""
     dims = int(spec.rotary_dim)
     i = torch.arange(dims // 2, dtype=torch.float64)
     f = float(spec.theta) ** (-2.0 * i / dims)
     magnitude = 1.0
-    if spec.factor is not None:
+    if spec.factor is not None and spec.low is not None:
+        turns = float(spec.original) * f / (2.0 * math.pi)     # how often a pair turns within ``original`` positions
+        low, high = float(spec.low), float(spec.high)
+        s = (turns - low) / (high - low) if high != low else torch.zeros_like(f)
+        blend = (1.0 - s) * f / float(spec.factor) + s * f
+        f = torch.where(turns > high, f, torch.where(turns < low, f / float(spec.factor), blend))
+    elif spec.factor is not None:
         def pair_at(turns):
             return dims * math.log(float(spec.original) / (2.0 * math.pi * float(turns))) / (2.0 * math.log(float(spec.theta)))
         lo = max(math.floor(pair_at(spec.fast)), 0)
@@ -88,8 +95,8 @@ class PairRotary:
 
 class ScaledHalfRotary:
     """Kind "rope_half_scaled": column i of the first ``rotary_dim`` turns with column i + rotary_dim/2; frequencies
-    stretched by wavelength when the spec gives a factor (see ScaledHalfRopeSpec).  No table: ``half_rotary`` hands the
-    kernels 32-bit frequencies, and they take angle = position * frequency, sine and cosine in 32-bit."""
+    stretched by wavelength when the spec gives a factor (see ScaledHalfRopeSpec).  No table: the kernels read
+    32-bit ``frequencies`` and take angle = position * frequency, sine and cosine in 32-bit, times ``magnitude``."""
 
     @staticmethod
     def weight_shapes(spec):
@@ -105,10 +112,6 @@ class ScaledHalfRotary:
 
     def prepare(self, n_positions: int) -> None:
         pass
-
-    def half_rotary(self):
-        """(frequencies [rotary_dim / 2] 32-bit, rotary_dim, what multiplies cosines and sines)."""
-        return self.frequencies, self.rotary_dim, self.magnitude
 
 
 class SinusoidEmbedding:

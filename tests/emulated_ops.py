@@ -208,26 +208,16 @@ class EmulatedOps:
         u = torch.einsum("s,rsw->rw", read_w.float(), X)
         return (u * torch.rsqrt((u * u).mean(-1, keepdim=True) + eps) * weight.float()).to(out_dtype)
 
-    def rotate_half_store(self, ctx, q, k, v, layer_cache, freqs, rot, magnitude):
+    def rotate_store(self, ctx, q, k, v, layer_cache, freqs, rot, magnitude, halves):
         group = layer_cache.group
         slots, pos = self._positions(ctx)
-
-        def turn(t):
-            t = t.float()
-            if freqs is None or not rot:
-                return t
-            angle = pos.float()[:, None] * freqs.float()[None, :]
-            c, s = (torch.cos(angle) * magnitude)[:, None, :], (torch.sin(angle) * magnitude)[:, None, :]
-            a, b = t[..., :rot // 2], t[..., rot // 2:rot]
-            return torch.cat([a * c - b * s, b * c + a * s, t[..., rot:]], dim=-1)
-
         page, off = self._physical(group, slots, pos)
         if bool((page < 0).any()):
             ctx.status |= 2
         ok = page >= 0
-        layer_cache.k[page[ok], :, off[ok]] = turn(k)[ok].to(layer_cache.k.dtype)
+        layer_cache.k[page[ok], :, off[ok]] = self._turn(k.float(), pos, freqs, rot, magnitude, halves)[ok].to(layer_cache.k.dtype)
         layer_cache.v[page[ok], :, off[ok]] = v.reshape(v.shape[0], group.v_heads, group.v_dim)[ok].to(layer_cache.v.dtype)
-        return turn(q).to(q.dtype)
+        return self._turn(q.float(), pos, freqs, rot, magnitude, halves).to(q.dtype)
 
     def diff_combine(self, a, heads, kv_heads, v_dim, lam, eps, post, gate=None):
         rows, per = a.shape[0], heads // kv_heads
@@ -363,20 +353,32 @@ class EmulatedOps:
         gf = g.float()
         return (o.reshape(rows, H * V) * (gf * torch.sigmoid(gf))).to(q.dtype)
 
-    def moe_route(self, h, router, correction, top, scale, bias=None, over_chosen=False):
-        z = h.float() @ router.float().T
+    def moe_route(self, h, router, correction, top, scale, bias=None, over_chosen=False, scores="softmax", groups=1, keep_groups=1,
+                  extra=0):
+        n_out = router.shape[0] - extra
+        full = h.float() @ router.float().T
+        z, behind = full[:, :n_out], full[:, n_out:]
         if bias is not None:
             z = z + bias.float()
         if over_chosen:
             chosen = torch.topk(z if correction is None else z + correction.float(), top, dim=-1).indices
             return chosen.to(torch.int32), torch.softmax(torch.gather(z, 1, chosen), dim=-1) * scale
-        s = torch.softmax(z, dim=-1)
-        chosen = torch.topk(s if correction is None else s + correction.float(), top, dim=-1).indices
+        s = torch.sigmoid(z) if scores == "sigmoid" else torch.softmax(z, dim=-1)
+        choice = s if correction is None else s + correction.float()
+        if groups > 1:
+            parts = choice.reshape(h.shape[0], groups, -1)
+            total = torch.topk(parts, min(2, parts.shape[-1]), dim=-1).values.sum(-1)
+            kept = torch.zeros_like(total, dtype=torch.bool).scatter(1, torch.topk(total, keep_groups, dim=-1).indices, True)
+            choice = parts.masked_fill(~kept[:, :, None], float("-inf")).reshape(choice.shape)
+        chosen = torch.topk(choice, top, dim=-1).indices
         picked = torch.gather(s, 1, chosen)
-        return chosen.to(torch.int32), picked / (picked.sum(-1, keepdim=True) + 1e-20) * scale
+        weight = picked / (picked.sum(-1, keepdim=True) + 1e-20) * scale
+        return (chosen.to(torch.int32), weight, behind) if extra else (chosen.to(torch.int32), weight)
 
-    def moe_experts(self, h, chosen, weight, w_gate_up, w_down, n_experts, alpha, limit, base):
+    def moe_experts(self, h, chosen, weight, w_gate_up, w_down, n_experts, alpha, limit, base, base_gate=None):
         out = torch.zeros(h.shape, dtype=torch.float32, device=h.device) if base is None else base.float().clone()
+        if base_gate is not None:
+            out = out * torch.sigmoid(base_gate)
         for r in range(h.shape[0]):
             for e, w in zip(chosen[r].tolist(), weight[r]):
                 if e >= n_experts:
@@ -386,6 +388,54 @@ class EmulatedOps:
                     act = self.swiglu(gu) if alpha is None else self.gated_clamp(gu, alpha, limit)
                     out[r] += w * self.linear(act, w_down[e])[0].float()
         return out.to(h.dtype)
+
+    # ---- a recurrence that decays by one number per head ----------------------------------
+
+    def conv_silu(self, ctx, u, weight, bias, state):
+        taps = weight.shape[0]
+        y = bias.float()[None, :].repeat(u.shape[0], 1)
+        for b in range(ctx.n_seqs):
+            slot, r0, r1 = int(ctx.seq_slot[b]), int(ctx.cu_q[b]), int(ctx.cu_q[b + 1])
+            past = state[slot].float() if taps > 1 else y.new_zeros((0, u.shape[1]))
+            hist = torch.cat([past, u[r0:r1].float()], dim=0)
+            for j in range(taps):
+                y[r0:r1] += weight[j].float()[None, :] * hist[j:j + (r1 - r0)]
+            if taps > 1:
+                state[slot] = hist[hist.shape[0] - (taps - 1):]
+        return (y * torch.sigmoid(y)).to(u.dtype)
+
+    def decay_scan(self, ctx, p, q_col, k_col, v_col, state, heads, kv_heads, dim, vdim, decay=None, step=None, skip=None, silu=False):
+        H, G, D, V = heads, kv_heads, dim, vdim
+        rows = p.shape[0]
+        act = (lambda t: t * torch.sigmoid(t)) if silu else (lambda t: t)
+        q = act(p[:, q_col:q_col + G * D].float()).reshape(rows, G, D).repeat_interleave(H // G, dim=1)
+        k = act(p[:, k_col:k_col + G * D].float()).reshape(rows, G, D).repeat_interleave(H // G, dim=1)
+        v = act(p[:, v_col:v_col + H * V].float()).reshape(rows, H, V)
+        if decay is not None:
+            a, w = decay[0][None, :].repeat(rows, 1), torch.ones(rows, H, device=p.device)
+        else:
+            dt, dt_bias, rate = step
+            w = torch.nn.functional.softplus(dt + dt_bias, threshold=80.0)
+            a = torch.exp(-rate * w)
+        out = torch.empty(rows, H, V, dtype=torch.float32, device=p.device)
+        cu = ctx.cu_q.tolist()
+        for b in range(ctx.n_seqs):
+            slot = int(ctx.seq_slot[b])
+            S = state[slot].reshape(H, D, V).clone()
+            for t in range(cu[b], cu[b + 1]):
+                S = a[t][:, None, None] * S + (w[t][:, None] * k[t])[:, :, None] * v[t][:, None, :]
+                out[t] = torch.einsum("hk,hkv->hv", q[t], S)
+            state[slot] = S.reshape(-1)
+        if skip is not None:
+            out = out + skip[None, :, None] * v
+        return out.reshape(rows, H * V)
+
+    def norm_gate(self, o, gate, weight, parts, eps, gate_first=False):
+        g = gate.float()
+        t = o * (g * torch.sigmoid(g)) if gate_first else o
+        t = t.reshape(o.shape[0], parts, -1)
+        y = (t * torch.rsqrt((t * t).mean(-1, keepdim=True) + eps)).reshape(o.shape) * weight
+        return (y if gate_first else y * torch.sigmoid(g)).to(gate.dtype)
 
     # ---- layer norms, the gated gelu, the delta rule with a decay per key channel ----------
 
