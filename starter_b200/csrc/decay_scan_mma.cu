@@ -33,7 +33,7 @@ __device__ __forceinline__ void split_pair(float x, float y, unsigned int& hi, u
 }
 
 // What a chunk's tokens need of the decays: c (as hi + lo, base 2), w, exp2(c), and exp2(c_last - c) w.
-struct ChunkDecays {
+struct alignas(16) ChunkDecays {   // read two numbers at a time
     float hi[DM_L], lo[DM_L], w[DM_L], grown[DM_L], left[DM_L];
     float total;   // exp2(c_last)
 };

@@ -1487,8 +1487,8 @@ class Ops:
         n_out = router.shape[0] - extra
         if scores not in ("softmax", "sigmoid") or (scores == "sigmoid" and over_chosen):
             raise KernelError(f"moe_route: scores are 'softmax' or (not over the chosen logits alone) 'sigmoid', got {scores!r}")
-        for extra in (correction, bias):
-            if extra is not None and (extra.dtype != torch.float32 or extra.numel() != n_out or not extra.is_contiguous()):
+        for t in (correction, bias):
+            if t is not None and (t.dtype != torch.float32 or t.numel() != n_out or not t.is_contiguous()):
                 raise KernelError(f"moe_route: correction and bias are {n_out} 32-bit numbers")
         if (router.dtype != torch.float32 or router.shape[1] != width or not h.is_contiguous()
                 or not router.is_contiguous() or n_out > 1024 or top > 32):
