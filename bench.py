@@ -517,9 +517,33 @@ SIPARAX_SIZES = {
     "2048": (_siparax_raw(2048, dict(heads=16, dim=128, rot_dim=64, vdim=128, q_rank=768, kv_rank=512),
                           dict(heads=32, kv_heads=32, dim=64, vdim=64, decay_rank=64, gate_rank=64), ff=8192), FAMILY_SIZES["2048"][0]),
 }
+def _nifalorn_raw(width, lightning, mamba, attention, experts, expert_ff, top, shared_ff, vocab=32000):
+    """A Nifalorn configuration of six layers: lightning attention or Mamba-2, then two attentions, twice."""
+    decay = [1.0 - 2.0 ** -(1.0 + 7.0 * i / (lightning["heads"] - 1)) for i in range(lightning["heads"])]
+    attn = {"type": "attention", "mixer": dict(attention, scale=attention["dim"] ** -0.5, diff=0.4,
+                                               rot={"base": 500000.0, "dims": attention["dim"],
+                                                    "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 4096}})}
+    kinds = [{"type": "lightning", "mixer": dict(lightning, decay=decay)}, attn, attn, {"type": "mamba2", "mixer": dict(mamba, conv=4)}, attn, attn]
+    mlp = {"kind": "moe", "router": {"experts": experts, "top": top, "scale": 2.0, "groups": {"count": 4, "keep": 2}},
+           "expert": {"ff": expert_ff}, "shared": {"ff": shared_ff}}
+    return {"architecture": "Nifalorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0},
+            "logit_scale": 1.0, "layers": [dict(kind, mlp=mlp) for kind in kinds]}
+
+
+# Nifalorn beside Nazulorn (the closest design the library has: a recurrence with a matrix state, attention with two score
+# maps of a bounded reach, a mixture of experts with a shared expert, scaled embedding and logits) at the same width,
+# layers, vocabulary, head counts, reach and expert sizes.
+NIFALORN_SIZES = {
+    "1024": (_nifalorn_raw(1024, dict(heads=8, dim=64, vdim=128), dict(heads=16, vdim=64, state=128, groups=2, norm_groups=2),
+                           dict(heads=8, kv_heads=2, dim=64, vdim=64, mask={"size": 1024}), experts=16, expert_ff=512, top=4,
+                           shared_ff=2048), NAZULORN_SIZES["1024"][0]),
+    "2048": (_nifalorn_raw(2048, dict(heads=16, dim=64, vdim=128), dict(heads=32, vdim=64, state=128, groups=4, norm_groups=4),
+                           dict(heads=8, kv_heads=4, dim=128, vdim=128, mask={"size": 2048}), experts=32, expert_ff=1024, top=4,
+                           shared_ff=4096), NAZULORN_SIZES["2048"][0]),
+}
 FAMILIES = {"kudazen": (FAMILY_SIZES, "qwen3", "Qwen3ForCausalLM"), "nazulorn": (NAZULORN_SIZES, "kudazen", "Kudazen"),
             "gulazen": (GULAZEN_SIZES, "nazulorn", "Nazulorn"), "paditar": (PADITAR_SIZES, "nazulorn", "Nazulorn"),
-            "siparax": (SIPARAX_SIZES, "kudazen", "Kudazen")}
+            "siparax": (SIPARAX_SIZES, "kudazen", "Kudazen"), "nifalorn": (NIFALORN_SIZES, "nazulorn", "Nazulorn")}
 
 
 class TimedOps:
@@ -583,6 +607,12 @@ class TimedOps:
             q, heads, dim, vdim = args[1], args[12], args[13], args[14]
             flops = 6.0 * q.shape[0] * heads * dim * vdim
             nbytes = 2 * args[0].n_seqs * heads * dim * vdim * 4 + q.shape[0] * heads * (2 * dim * 2 + 3 * vdim * 2 + dim * 4)
+        elif name == "decay_scan":
+            p, heads, kv_heads, dim, vdim = args[1], args[6], args[7], args[8], args[9]
+            flops = 4.0 * p.shape[0] * heads * dim * vdim         # the write and the read
+            nbytes = (2 * args[0].n_seqs * heads * dim * vdim * 4 + p.shape[0] * (2 * kv_heads * dim + heads * vdim) * 2 + self._nbytes([out]))
+        elif name == "conv_silu":
+            nbytes = self._nbytes([args[1], args[2], args[3], out])
         elif name == "delta_scan":
             qkv, z, heads, dim, vdim = args[1], args[2], args[10], args[12], args[13]
             flops = 7.0 * qkv.shape[0] * heads * dim * vdim       # decay, what the key holds, the write, the read
@@ -717,9 +747,9 @@ def _family_arm(torch, raw, peaks, prefill_tokens, batch, context, steps, warmup
 
 
 def run_family(args) -> int:
-    """--family kudazen | nazulorn | gulazen | paditar | siparax: the design at a few sizes that resemble a real model's layers (random weights),
+    """--family kudazen | nazulorn | gulazen | paditar | siparax | nifalorn: the design at a few sizes that resemble a real model's layers (random weights),
     beside the library's closest model of the same width, feed-forward work per token, layer count and vocabulary (Kudazen
-    beside the Qwen3 decoder, Nazulorn and Siparax beside Kudazen, Gulazen and Paditar beside Nazulorn).  One JSON line."""
+    beside the Qwen3 decoder, Nazulorn and Siparax beside Kudazen, Gulazen, Paditar and Nifalorn beside Nazulorn).  One JSON line."""
     import torch
     peaks, peak_source = load_peaks()
     torch.cuda.set_device(0)
@@ -947,10 +977,10 @@ def main() -> int:
     ap.add_argument("--context", type=int, default=0)
     ap.add_argument("--skip-points", action="store_true", help="leave out the further decode points")
     ap.add_argument("--skip-e2e", action="store_true")
-    ap.add_argument("--family", default="", choices=["", "kudazen", "nazulorn", "gulazen", "paditar", "siparax"],
+    ap.add_argument("--family", default="", choices=["", "kudazen", "nazulorn", "gulazen", "paditar", "siparax", "nifalorn"],
                     help="instead of the default workload: this model family at a few layer sizes, beside the library's closest "
-                         "model of equal size (kudazen beside the Qwen3 shape, nazulorn and siparax beside kudazen, gulazen and paditar "
-                         "beside nazulorn)")
+                         "model of equal size (kudazen beside the Qwen3 shape, nazulorn and siparax beside kudazen, gulazen, paditar and "
+                         "nifalorn beside nazulorn)")
     ap.add_argument("--sizes", default="", help="with --family: sizes to run, with commas between them (default: all)")
     args = ap.parse_args()
 
