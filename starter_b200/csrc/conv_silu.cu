@@ -21,6 +21,17 @@ template <> __device__ __forceinline__ void channels_load<__nv_bfloat16, 8>(cons
         v[2 * e + 1] = f.y;
     }
 }
+template <> __device__ __forceinline__ void channels_load<float, 8>(const float* p, float (&v)[8]) {
+    const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+    v[0] = a.x;
+    v[1] = a.y;
+    v[2] = a.z;
+    v[3] = a.w;
+    v[4] = b.x;
+    v[5] = b.y;
+    v[6] = b.z;
+    v[7] = b.w;
+}
 template <class T, int VEC> __device__ __forceinline__ void channels_store(T* p, const float (&v)[VEC]) {
 #pragma unroll
     for (int i = 0; i < VEC; ++i) p[i] = from_f<T>(v[i]);
@@ -87,8 +98,8 @@ conv_silu_kernel(const T* __restrict__ u, long long ld, const float* __restrict_
 #pragma unroll
             for (int i = 0; i < VEC; ++i) {
                 y[i] = fmaf(wj[i], x[i], y[i]);
-                if (ADVANCE && j > 0) rec[(long long)(j - 1) * C + c + i] = x[i];   // entry j - 1 was read in an earlier turn
             }
+            if (ADVANCE && j > 0) channels_store<float, VEC>(rec + (long long)(j - 1) * C + c, x);   // entry j - 1 was read in an earlier turn
         }
 #pragma unroll
         for (int i = 0; i < VEC; ++i) y[i] = silu_value(y[i]);
@@ -105,8 +116,9 @@ int sb_conv_silu(int dtype, const void* u, long long ld, const float* w, const f
     if (taps < 1 || (taps > 1 && state == nullptr) || C < 1) return (int)cudaErrorInvalidValue;
     typedef __nv_bfloat16 bf;
     const bool many = batch.n_rows >= 256 && !one_row;
-    const bool vec = dtype == SB_BF16 && batch.n_rows >= 64 && C % 8 == 0 && ld % 8 == 0 && (reinterpret_cast<size_t>(u) & 15) == 0;
-    const int R = many ? 8 : 1;
+    const size_t bases = reinterpret_cast<size_t>(u) | reinterpret_cast<size_t>(w) | reinterpret_cast<size_t>(bias) | reinterpret_cast<size_t>(state);
+    const bool vec = dtype == SB_BF16 && batch.n_rows >= 64 && C % 8 == 0 && ld % 8 == 0 && state_slot % 4 == 0 && (bases & 15) == 0;
+    const int R = many ? 4 : 1;
     const int lanes = vec ? C / 8 : C, threads = lanes >= 128 ? 128 : (lanes + 31) / 32 * 32;
     const dim3 grid((batch.n_rows + R - 1) / R, (lanes + threads - 1) / threads);
     if (grid.y > 65535) return (int)cudaErrorInvalidValue;
@@ -117,10 +129,10 @@ int sb_conv_silu(int dtype, const void* u, long long ld, const float* w, const f
     do {                                                    \
         if (one_row && taps > 1) SB_CS(T, VEC, 1, 0, true); \
         else if (R == 1) SB_CS(T, VEC, 1, 0, false);        \
-        else if (taps == 4) SB_CS(T, VEC, 8, 4, false);     \
-        else if (taps == 3) SB_CS(T, VEC, 8, 3, false);     \
-        else if (taps == 2) SB_CS(T, VEC, 8, 2, false);     \
-        else SB_CS(T, VEC, 8, 0, false);                    \
+        else if (taps == 4) SB_CS(T, VEC, 4, 4, false);     \
+        else if (taps == 3) SB_CS(T, VEC, 4, 3, false);     \
+        else if (taps == 2) SB_CS(T, VEC, 4, 2, false);     \
+        else SB_CS(T, VEC, 4, 0, false);                    \
     } while (0)
     if (dtype == SB_F32) SB_CST(float, 1);
     else if (vec) SB_CST(bf, 8);

@@ -33,5 +33,5 @@ struct SbDecay {
     int V;
 };
 
-__device__ __forceinline__ float silu_value(float x) { return x / (1.0f + expf(-x)); }
+__device__ __forceinline__ float silu_value(float x) { return __fdividef(x, 1.0f + expf(-x)); }
 __device__ __forceinline__ float softplus_value(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }

@@ -9,6 +9,11 @@
 // the weighted keys) is written as two bfloat16 numbers hi + lo, so that it keeps 16 bits; queries, keys and values are
 // bfloat16 numbers and lose nothing.  Log-decays are summed in 64-bit and kept as two 32-bit numbers, so that a chunk
 // with strong decays keeps the differences between its weak ones.
+//
+// A step with few sequences and heads leaves most SMs without a block when every block walks a whole sequence.  The chunks
+// are then dealt out in runs: decay_chunk_kernel<.., STATES> takes every run from a zero state and leaves what it adds and how
+// far it decays, decay_runs_kernel walks the runs in order (one multiplication and one addition per entry of the state) and
+// leaves the state at each run's start, and decay_chunk_kernel<.., OUTPUTS> takes the outputs of all runs side by side.
 #include "decay_scan.cuh"
 #include "mma_utils.cuh"
 
@@ -79,12 +84,24 @@ __device__ __forceinline__ void chunk_decays(const SbDecay& a, int head, int row
     if (lane == 0) c.total = exp2f((float)last);
 }
 
-// A block of four warps per (sequence, head, DM_VB value columns) walks the sequence's chunks.  Products with the queries:
+enum { DM_WHOLE = 0, DM_STATES = 1, DM_OUTPUTS = 2 };
+
+// The runs of a step: `count` per sequence of `chunks` chunks each; states [sequence][run][head][D][V] and how far each run
+// decays, [sequence][run][head].
+struct ChunkRuns {
+    float* states;
+    float* decays;
+    int count;
+    int chunks;
+};
+
+// A block of four warps per (sequence and run, head, DM_VB value columns) walks the run's chunks (DM_WHOLE: one run per
+// sequence, from and back into its record).  Products with the queries:
 // warp w owns the tokens 16 w .. 16 w + 15 of the chunk.  State: warp w owns a quarter of the key channels (DP 32: half of
 // the channels and half of the columns).  DP: the key channels rounded up to 32, 64, 128 or 256.
-template <int DP>
+template <int DP, int MODE>
 __global__ void __launch_bounds__(DM_THREADS, DP <= 128 ? 2 : 1)
-decay_chunk_kernel(SbDecay a, SbBatch batch, float* __restrict__ out, int vec) {
+decay_chunk_kernel(SbDecay a, SbBatch batch, float* __restrict__ out, int vec, ChunkRuns runs) {
     typedef __nv_bfloat16 bf;
     constexpr int QLD = DP + 8, STAGE = 2 * DM_L * QLD + DM_L * DM_VLD;
     constexpr int MT = DP >= 64 ? DP / 64 : 1, NT = DP >= 64 ? 4 : 2;    // a warp's tiles of 16 channels and of 8 columns of the state
@@ -94,11 +111,17 @@ decay_chunk_kernel(SbDecay a, SbBatch batch, float* __restrict__ out, int vec) {
     bf* Sl = Sh + DP * DM_VLD;
     __shared__ ChunkDecays decays[2];
     const int D = a.D, V = a.V, H = a.H;
-    const int s = blockIdx.x, head = blockIdx.y, col0 = blockIdx.z * DM_VB, nv = min(DM_VB, V - col0);
+    const int s = MODE == DM_WHOLE ? blockIdx.x : blockIdx.x / runs.count, run = MODE == DM_WHOLE ? 0 : blockIdx.x % runs.count;
+    const int head = blockIdx.y, col0 = blockIdx.z * DM_VB, nv = min(DM_VB, V - col0);
     const int tid = threadIdx.x, lane = tid & 31, w = tid >> 5, g = lane >> 2, t = lane & 3;
     const float skip = a.skip != nullptr ? a.skip[head] : 0.f;
     pdl_wait();
-    const int row0 = batch.cu_q[s], n = batch.cu_q[s + 1] - row0, chunks = (n + DM_L - 1) / DM_L;
+    int row0 = batch.cu_q[s], n = batch.cu_q[s + 1] - row0;
+    if (MODE != DM_WHOLE) {                                 // the run's own rows
+        row0 += run * runs.chunks * DM_L;
+        n = min(n - run * runs.chunks * DM_L, runs.chunks * DM_L);
+    }
+    const int chunks = (n + DM_L - 1) / DM_L;
     if (n <= 0) return;
     const int grp = head / (H / a.G);
     const bf* base = (const bf*)a.p;
@@ -113,7 +136,7 @@ decay_chunk_kernel(SbDecay a, SbBatch batch, float* __restrict__ out, int vec) {
                 const int r = e / QC, c = (e % QC) * 8;
                 const bool ok = r < nt && c < D;
                 const bf* src = base + (ok ? (first + r) * a.ld + grp * D + c : 0);
-                cp_async_16_or_none(Q + r * QLD + c, src + (ok ? a.q_col : 0), ok);
+                if (MODE != DM_STATES) cp_async_16_or_none(Q + r * QLD + c, src + (ok ? a.q_col : 0), ok);
                 cp_async_16_or_none(K + r * QLD + c, src + (ok ? a.k_col : 0), ok);
             }
             for (int e = tid; e < DM_L * VC; e += DM_THREADS) {
@@ -127,7 +150,7 @@ decay_chunk_kernel(SbDecay a, SbBatch batch, float* __restrict__ out, int vec) {
                 const int r = e / DP, c = e % DP;
                 const bool ok = r < nt && c < D;
                 const bf* src = base + (first + r) * a.ld + grp * D + c;
-                Q[r * QLD + c] = ok ? src[a.q_col] : zero;
+                if (MODE != DM_STATES) Q[r * QLD + c] = ok ? src[a.q_col] : zero;
                 K[r * QLD + c] = ok ? src[a.k_col] : zero;
             }
             for (int e = tid; e < DM_L * DM_VB; e += DM_THREADS) {
@@ -139,7 +162,9 @@ decay_chunk_kernel(SbDecay a, SbBatch batch, float* __restrict__ out, int vec) {
     };
 
     const int m_base = DP >= 64 ? w * MT * 16 : (w & 1) * 16, n_base = DP >= 64 ? 0 : (w >> 1) * 16;
-    float* Sg = a.state + (long long)batch.seq_slot[s] * a.state_slot + (long long)head * D * V + col0;
+    const long long cell = ((long long)blockIdx.x * H + head);     // the run's place among the runs of the step
+    float* Sg = (MODE == DM_WHOLE ? a.state + (long long)batch.seq_slot[s] * a.state_slot + (long long)head * D * V
+                                  : runs.states + cell * D * V) + col0;
     float S[MT][NT][4];
 #pragma unroll
     for (int mt = 0; mt < MT; ++mt)
@@ -148,8 +173,9 @@ decay_chunk_kernel(SbDecay a, SbBatch batch, float* __restrict__ out, int vec) {
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 const int d = m_base + mt * 16 + g + (e >> 1) * 8, c = n_base + nt * 8 + 2 * t + (e & 1);
-                S[mt][nt][e] = d < D && c < nv ? Sg[(long long)d * V + c] : 0.f;
+                S[mt][nt][e] = MODE != DM_STATES && d < D && c < nv ? Sg[(long long)d * V + c] : 0.f;
             }
+    float decayed = 1.f;                                    // how far the run has decayed
     auto publish = [&]() {
 #pragma unroll
         for (int mt = 0; mt < MT; ++mt)
@@ -166,7 +192,7 @@ decay_chunk_kernel(SbDecay a, SbBatch batch, float* __restrict__ out, int vec) {
     };
     fetch(0);
     if (w == 0) chunk_decays(a, head, row0, min(DM_L, n), decays[0]);
-    publish();
+    if (MODE != DM_STATES) publish();
 
     for (int ch = 0; ch < chunks; ++ch) {
         cp_async_wait<0>();
@@ -179,8 +205,8 @@ decay_chunk_kernel(SbDecay a, SbBatch batch, float* __restrict__ out, int vec) {
         const bf* K = Q + DM_L * QLD;
         const bf* Vs = K + DM_L * QLD;
         const ChunkDecays& dc = decays[ch & 1];
+        if (MODE != DM_STATES) {
         const int i0 = w * 16 + g;              // this thread's tokens: i0 and i0 + 8
-
         float sc[8][4], o[4][4];
 #pragma unroll
         for (int i = 0; i < 8; ++i)
@@ -278,8 +304,11 @@ decay_chunk_kernel(SbDecay a, SbBatch batch, float* __restrict__ out, int vec) {
                 }
             }
         }
+        }
+        if (MODE == DM_OUTPUTS && ch + 1 == chunks) break;   // nobody asks for the state after the run
         // the state after the chunk
         const float total = dc.total;
+        decayed *= total;
 #pragma unroll
         for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
@@ -316,11 +345,13 @@ decay_chunk_kernel(SbDecay a, SbBatch batch, float* __restrict__ out, int vec) {
                 }
             }
         }
-        if (ch + 1 < chunks) {
+        if (MODE != DM_STATES && ch + 1 < chunks) {
             __syncthreads();                    // nobody reads the state of this chunk's start any more
             publish();
         }
     }
+    if (MODE == DM_OUTPUTS) return;
+    if (MODE == DM_STATES && tid == 0 && blockIdx.z == 0) runs.decays[cell] = decayed;
 #pragma unroll
     for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
@@ -332,30 +363,74 @@ decay_chunk_kernel(SbDecay a, SbBatch batch, float* __restrict__ out, int vec) {
             }
 }
 
-template <int DP>
-static int launch_decay_chunk(SbDecay a, SbBatch batch, float* out, int vec, cudaStream_t stream) {
+// One thread per entry of a sequence's state: every run's place receives the state at its start, the record the state after
+// the last run.  Eight runs' contributions are fetched ahead of the chain.
+__global__ void __launch_bounds__(256) decay_runs_kernel(SbDecay a, SbBatch batch, ChunkRuns runs) {
+    pdl_wait();
+    const int s = blockIdx.x, head = blockIdx.y, size = a.D * a.V;
+    const int at = blockIdx.z * blockDim.x + threadIdx.x;
+    if (at >= size) return;
+    const int n = batch.cu_q[s + 1] - batch.cu_q[s], per = runs.chunks * DM_L, count = min(runs.count, (n + per - 1) / per);
+    float* rec = a.state + (long long)batch.seq_slot[s] * a.state_slot + (long long)head * size + at;
+    float S = *rec;
+    for (int r0 = 0; r0 < count; r0 += 8) {
+        float add[8], keep[8];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            const long long cell = ((long long)s * runs.count + min(r0 + i, count - 1)) * a.H + head;
+            add[i] = runs.states[cell * size + at];
+            keep[i] = runs.decays[cell];
+        }
+#pragma unroll
+        for (int i = 0; i < 8; ++i)
+            if (r0 + i < count) {
+                runs.states[(((long long)s * runs.count + r0 + i) * a.H + head) * size + at] = S;
+                S = fmaf(keep[i], S, add[i]);
+            }
+    }
+    if (count > 0) *rec = S;
+}
+
+template <int DP, int MODE>
+static int launch_chunk_walk(SbDecay a, SbBatch batch, float* out, int vec, ChunkRuns runs, cudaStream_t stream) {
     const size_t smem = (size_t)(2 * (2 * DM_L * (DP + 8) + DM_L * DM_VLD) + 2 * DP * DM_VLD) * sizeof(__nv_bfloat16);
-    const cudaError_t err = cudaFuncSetAttribute(decay_chunk_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    const cudaError_t err = cudaFuncSetAttribute(decay_chunk_kernel<DP, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (err != cudaSuccess) return (int)err;
-    const dim3 grid(batch.n_seqs, a.H, (a.V + DM_VB - 1) / DM_VB);
+    const dim3 grid(batch.n_seqs * (MODE == DM_WHOLE ? 1 : runs.count), a.H, (a.V + DM_VB - 1) / DM_VB);
     if (grid.z > 65535) return (int)cudaErrorInvalidValue;
-    sb_launch(decay_chunk_kernel<DP>, grid, DM_THREADS, smem, stream, a, batch, out, vec);
+    sb_launch(decay_chunk_kernel<DP, MODE>, grid, DM_THREADS, smem, stream, a, batch, out, vec, runs);
     SB_LAUNCH_CHECK();
+}
+
+template <int DP>
+static int launch_decay_chunk(SbDecay a, SbBatch batch, float* out, int vec, ChunkRuns runs, cudaStream_t stream) {
+    if (runs.count <= 1) return launch_chunk_walk<DP, DM_WHOLE>(a, batch, out, vec, runs, stream);
+    const int err = launch_chunk_walk<DP, DM_STATES>(a, batch, out, vec, runs, stream);
+    if (err) return err;
+    const dim3 grid(batch.n_seqs, a.H, (a.D * a.V + 255) / 256);
+    if (grid.z > 65535) return (int)cudaErrorInvalidValue;
+    sb_launch(decay_runs_kernel, grid, 256, 0, stream, a, batch, runs);
+    return launch_chunk_walk<DP, DM_OUTPUTS>(a, batch, out, vec, runs, stream);
 }
 
 extern "C" {
 
 // bfloat16 rows whose queries, keys and values are not to be activated any more; D up to 256; out [rows, H V] floats.
-int sb_decay_chunk(SbDecay a, SbBatch batch, float* out, cudaStream_t stream) {
+// n_runs > 1: runs of run_chunks chunks of 64 tokens (n_runs * run_chunks cover the longest sequence), with scratch for
+// n_seqs * n_runs * H states of D * V floats, and as many numbers.
+int sb_decay_chunk(SbDecay a, SbBatch batch, float* out, int n_runs, int run_chunks, float* run_states, float* run_decays,
+                   cudaStream_t stream) {
     if (batch.n_seqs <= 0 || batch.n_rows <= 0) return 0;
-    if (a.D < 1 || a.D > 256 || a.V < 1 || a.G < 1 || a.H % a.G || a.H > 65535 || a.act || (a.log2_decay == nullptr) == (a.dt == nullptr))
+    if (a.D < 1 || a.D > 256 || a.V < 1 || a.G < 1 || a.H % a.G || a.H > 65535 || a.act || (a.log2_decay == nullptr) == (a.dt == nullptr)
+        || (n_runs > 1 && (run_chunks < 1 || run_states == nullptr || run_decays == nullptr)))
         return (int)cudaErrorInvalidValue;
+    const ChunkRuns runs = {run_states, run_decays, n_runs, run_chunks};
     const int vec = a.ld % 8 == 0 && a.q_col % 8 == 0 && a.k_col % 8 == 0 && a.v_col % 8 == 0 && a.D % 8 == 0 && a.V % 8 == 0
                     && (reinterpret_cast<size_t>(a.p) & 15) == 0;
-    if (a.D <= 32) return launch_decay_chunk<32>(a, batch, out, vec, stream);
-    if (a.D <= 64) return launch_decay_chunk<64>(a, batch, out, vec, stream);
-    if (a.D <= 128) return launch_decay_chunk<128>(a, batch, out, vec, stream);
-    return launch_decay_chunk<256>(a, batch, out, vec, stream);
+    if (a.D <= 32) return launch_decay_chunk<32>(a, batch, out, vec, runs, stream);
+    if (a.D <= 64) return launch_decay_chunk<64>(a, batch, out, vec, runs, stream);
+    if (a.D <= 128) return launch_decay_chunk<128>(a, batch, out, vec, runs, stream);
+    return launch_decay_chunk<256>(a, batch, out, vec, runs, stream);
 }
 
 }  // extern "C"

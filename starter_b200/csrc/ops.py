@@ -183,7 +183,7 @@ class Ops:
             "sb_moe_combine": [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
                                c_int, c_void_p, c_int, c_void_p],
             "sb_decay_step": [c_int, SbDecay, SbBatch, c_void_p, c_int, c_void_p],
-            "sb_decay_chunk": [SbDecay, SbBatch, c_void_p, c_void_p],
+            "sb_decay_chunk": [SbDecay, SbBatch, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p],
             "sb_silu_columns": [c_int, c_void_p, c_longlong, c_int, c_int, c_void_p],
             "sb_norm_gate": [c_int, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_int, c_void_p],
             "sb_conv_silu": [c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_longlong, SbBatch, c_int, c_int, c_void_p,
@@ -1446,16 +1446,40 @@ class Ops:
                     _ptr(decay[1]) if decay is not None else None, _ptr(dt), dt.stride(0) if dt is not None else 0, _ptr(dt_bias), _ptr(rate),
                     _ptr(skip), _ptr(state), state.stride(0), H, G, D, V)
         if chunks:
-            self._check(self.lib.sb_decay_chunk(a, self._batch(ctx), _ptr(out), self._stream()), "decay_chunk")
+            runs, per_run = self.decay_runs(ctx.n_seqs, ctx.max_q_len, H, V)
+            states = decays = None
+            if runs > 1:
+                states = torch.empty(ctx.n_seqs * runs * H * D * V, dtype=torch.float32, device=p.device)
+                decays = torch.empty(ctx.n_seqs * runs * H, dtype=torch.float32, device=p.device)
+                self.launches += 2   # what the runs add, the walk over them, the outputs
+            self._check(self.lib.sb_decay_chunk(a, self._batch(ctx), _ptr(out), runs, per_run, _ptr(states), _ptr(decays), self._stream()),
+                        "decay_chunk")
         else:
-            self._check(self.lib.sb_decay_step(_code(p.dtype), a, self._batch(ctx), _ptr(out), self.decay_columns(ctx.n_seqs, H, V),
+            self._check(self.lib.sb_decay_step(_code(p.dtype), a, self._batch(ctx), _ptr(out), self.decay_columns(ctx.n_seqs, H, D, V),
                                                self._stream()), "decay_step")
         return out
 
-    def decay_columns(self, n_seqs: int, heads: int, vdim: int) -> int:
-        """Value columns per block of the token-by-token kernel: as many as leave two blocks per SM."""
+    force_decay_runs = None   # runs per sequence for tests and tuning; None = the rule below
+
+    def decay_runs(self, n_seqs: int, max_q_len: int, heads: int, vdim: int):
+        """(runs per sequence, chunks of 64 tokens per run) of a long step: as many runs as give every SM two blocks, two
+        chunks each at least; one run when whole sequences do already.  Measured on 2,048 tokens (us, 1 / 4 / 8 / 16 runs): 8
+        heads of 64 x 128: 113 / 48 / 31 / 34; 32 heads of 128 x 64: 155 / 76 / 80 / 86; four sequences of 64 such heads: 408 /
+        585 / 610 / 717."""
+        chunks = -(-max_q_len // 64)
+        blocks = n_seqs * heads * -(-vdim // 32)
+        want = self.force_decay_runs or min(2 * self.sm_count() // blocks, chunks // 2)
+        if want < 2 or chunks < 2:
+            return 1, chunks
+        per_run = -(-chunks // want)
+        return -(-chunks // per_run), per_run
+
+    def decay_columns(self, n_seqs: int, heads: int, dim: int, vdim: int) -> int:
+        """Value columns per block of the token-by-token kernel: as many as leave a thread four key channels or fewer and
+        every SM a block.  Measured on one token each (us, 32 / 64 / 128 columns): 8 sequences of 32 heads of 128 x 64: 6.8
+        / 8.0 / 8.2, 64 sequences: 40 / 48 / 50; 8 sequences of 16 heads of 64 x 128: 6.3 / 4.0 / 4.5."""
         for columns in (128, 64):
-            if vdim > columns // 2 and n_seqs * heads * -(-vdim // columns) >= 2 * self.sm_count():
+            if columns * dim <= 4096 and vdim > columns // 2 and n_seqs * heads * -(-vdim // columns) >= self.sm_count():
                 return columns
         return 32
 

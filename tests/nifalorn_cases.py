@@ -107,8 +107,13 @@ def config(name):
     return config_from_dict(copy.deepcopy(CASES[name]))
 
 
-def write_folder(name, folder, dtype=torch.bfloat16, shards=1):
-    return write_model_folder(config(name), SEEDS[name], folder, dtype=dtype, shards=shards)
+def write_folder(name, folder, dtype=torch.bfloat16, shards=1, steady=False):
+    """``steady``: corrections so far apart that they alone choose the experts, and no close call that rounding turns."""
+    cfg = config(name)
+    if steady:
+        ordinary = cfg.random_init
+        object.__setattr__(cfg, "random_init", lambda tensor, shape: (0.0, 6.0) if tensor.endswith("correction") else ordinary(tensor, shape))
+    return write_model_folder(cfg, SEEDS[name], folder, dtype=dtype, shards=shards)
 
 
 def plain_logits(folder, seqs):
